@@ -691,10 +691,18 @@ void b200_runner_set_tp_fused(b200_runner*, int32_t on);
  * POSTNORM.  The mixer's input may pass a token shift first (shift_w), and the layer may close with an average over
  * the results of all layers so far (depth_w); both are described at b200_hybrid_layer.                              */
 #define B200_LAYOUT_PRENORM 3
+/* HYPER: pre-norm sublayers inside hyper-connections.  The model keeps `streams` residual streams X_1 .. X_S (all equal to
+ * the embedding row at the start) instead of one; a sublayer reads a weighted sum of them and every stream is rewritten:
+ * y = sublayer(norm(sum_s in[s] X_s)), X_t <- sum_s mix[s][t] X_s + out[t] y (b200_hyper_step).  The model ends with the
+ * sum of the streams.  The feed-forward is chosen as in POSTNORM.  All layers of such a model have this layout.     */
+#define B200_LAYOUT_HYPER 4
+#define B200_MAX_STREAMS 16
 /* Norm kinds of the stream norms (norm_kind of a layer, final_norm_kind of the model).  RMS: x / sqrt(mean(x^2) + eps)
- * * (offset + w).  DYNTANH: tanh(alpha * x) * w + b, element by element, no mean or variance (eps is not used).   */
+ * * (offset + w).  DYNTANH: tanh(alpha * x) * w + b, element by element, no mean or variance (eps is not used).
+ * LAYER: (x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + w) + b.                                            */
 #define B200_NORM_RMS 0
 #define B200_NORM_DYNTANH 1
+#define B200_NORM_LAYER 2
 
 void b200_resid_rmsnorm(void* out, const float* x, const float* w, int32_t num_tokens, int32_t width, float eps,
                         float w_offset, int32_t dt, int64_t stream);
@@ -714,8 +722,26 @@ void b200_stream_norm(void* out, const float* x, const float* w, const float* bi
                       float eps, float w_offset, const uint32_t* rows, const float* shift_w, float* shift_state,
                       const int32_t* state_slots, const uint32_t* cu_seqlens_q, const uint32_t* context_lens,
                       int32_t num_seqs, int32_t num_tokens, int32_t width, int32_t dt, int64_t stream);
+/* One step of hyper-connections over `streams` residual streams of T rows: the update that closes a sublayer, fused with
+ * the read, norm and rounding that open the next one.  With X_s = x_in + s * in_stride (fp32 [T, width]; in_stride 0: all
+ * streams equal x_in's rows):
+ *   y != NULL or down != NULL:  Z_t = sum_s mix[s * streams + t] X_s + out_w[t] * y   (else Z = X)
+ *   x_out != NULL: stream t is stored at x_out + t * out_stride (x_out may be x_in with the same stride)
+ *   out   != NULL: out[r] = norm(sum_t in_w[t] Z_t) in dtype dt (in_w NULL: ones)
+ * mix, out_w, in_w, w, bias: fp32 on the device (bias may be NULL).  rows (u32 [T], may be NULL; then x_out is NULL): row r
+ * of out belongs to stream row rows[r].  The sublayer's rows are y fp32 [*, width] or, where `down` is given, the weighted
+ * sum of routed experts sum_j top_w[p] * down[slot_of_pair[p]], p = row * top + j (b200_moe_experts_rows).          */
+void b200_hyper_step(void* out, float* x_out, int64_t out_stride, const float* x_in, int64_t in_stride, const float* y,
+                     const float* down, const int32_t* slot_of_pair, const float* top_w, int32_t top, const float* mix,
+                     const float* out_w, const float* in_w, const float* w, const float* bias, float alpha, int32_t kind,
+                     float eps, float w_offset, const uint32_t* rows, int32_t streams, int32_t num_tokens, int32_t width,
+                     int32_t dt, int64_t stream);
+/* out [T, n] (dtype dt) = act(up + bias), up fp32 with row stride ld: act 1 relu(.)^2, 2 the exact GELU
+ * z/2 (1 + erf(z / sqrt 2)); bias fp32 [n] or NULL.                                                                 */
+void b200_ff_act(void* out, const float* up, int32_t ld, const float* bias, int32_t act, int32_t num_tokens, int32_t n,
+                 int32_t dt, int64_t stream);
 /* out fp32 [n] = sum over j < count of w[j] * hist[j * stride + i]: a weighted sum of `count` stored streams (w fp32
- * [count], on the device).  out may be one of the streams' successors but none of the `count` inputs.              */
+ * [count], on the device; NULL: ones).  out may be one of the streams' successors but none of the `count` inputs.              */
 void b200_depth_mix(float* out, const float* hist, int64_t stride, const float* w, int32_t count, int64_t n,
                     int64_t stream);
 /* Windowed softmax attention with grouped K / V heads (csrc/window_attn.cu).  proj fp32 [T, ld] = [q: heads x dim |
@@ -750,7 +776,8 @@ int64_t b200_window_attn_workspace_bytes_ex(int32_t num_tokens, int32_t heads, i
  *                     1 + coef * ln(floor((p + 1) / every) + 1)                       (after norm and rotation)
  *   dist_slopes fp32 [heads] or NULL: the score of query position i against key position j is lowered by slope_h * (i - j)
  *                     (after scale and cap)
- *   gate_elems  != 0: the output gate has heads x vdim logits per token (one per output element) instead of heads   */
+ *   gate_elems  != 0: the output gate has heads x vdim logits per token (one per output element) instead of heads
+ * head_norm == 2: every head is RMS-normed on its own and there is no weight (q_norm_w / k_norm_w are not read)      */
 typedef struct b200_attn_options {
   int32_t head_norm, v_from_k, q_temp_every, gate_elems;
   float q_temp_coef;
@@ -770,6 +797,17 @@ typedef struct b200_attn_options {
   float rot_mag;
   const double* v_rot_freq;
   int32_t v_heads, chunk, out_f32, no_cache;
+  /* (fields below: NULL / zero = off)
+   *   dist_bias   fp32 [heads, dist_n]: the score of query position i against key position j gains
+   *                     dist_bias[h, min(i - j, dist_n - 1)] (after scale and cap)
+   *   v_first_out (prep) fp32 [T, v_heads x vdim]: the value rows (projection + bias) are also stored here
+   *   v_first     (prep) fp32 [T, v_heads x vdim]: the value rows become (1 - v_mix) v + v_mix v_first before they are
+   *                     rotated and cached                                                                            */
+  const float* dist_bias;
+  int32_t dist_n;
+  float v_mix;
+  float* v_first_out;
+  const float* v_first;
 } b200_attn_options;
 /* What follows the softmax-weighted sums where more than a gate does: out [T, heads, vdim] (dtype dt) from a fp32
  * [T, maps * heads, vdim] (map after map).  maps == 2: o = a[map 0] - lambda * a[map 1] (differential attention).
@@ -885,6 +923,19 @@ void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, cons
                          int32_t width, int32_t ff, int32_t act, int32_t accumulate, const void* ident,
                          int32_t ident_f32, int32_t dt, void* workspace, int64_t stream);
 
+/* Router scores and weights beyond b200_moe_route_ex.  score 0: softmax over all outputs, 1: the sigmoid of every logit;
+ * group_top: a group's score is the sum of its group_top (1 or 2) largest choice scores; renorm != 0: the chosen weights
+ * are divided by their sum + 1e-20 (before `scale`).                                                                */
+void b200_moe_route_full(const float* logits, const float* bias, int32_t num_tokens, int32_t experts, int32_t top,
+                         int32_t groups, int32_t keep, int32_t score, int32_t group_top, int32_t renorm, float scale,
+                         int32_t* top_idx, float* top_w, int64_t stream);
+/* b200_moe_experts_ex without the weighted sum: *down receives the address (inside workspace) of the experts' output rows
+ * fp32 [T * top, width], *slot_of_pair that of the row of pair p = token * top + choice.  No identity experts.      */
+void b200_moe_experts_rows(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down,
+                           int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff, int32_t act,
+                           int32_t dt, void* workspace, const float** down, const int32_t** slot_of_pair,
+                           int64_t stream);
+
 typedef struct b200_hybrid_config {
   int32_t width, vocab, num_layers;
   int32_t dt;                               /* 0 = bf16 operands and cache, 1 = fp32 */
@@ -895,7 +946,8 @@ typedef struct b200_hybrid_config {
   float embed_scale;                        /* the embedding row is multiplied by it */
   float embed_pos_base;                     /* > 0: a sinusoidal position vector joins the embedding row: entry 2i is
                                                sin(p base^(-2i / width)), entry 2i + 1 the cosine of the same angle */
-  int32_t final_norm_kind;                  /* B200_NORM_*; DYNTANH: see b200_hybrid_set_final_norm */
+  int32_t final_norm_kind;                  /* B200_NORM_*; DYNTANH, LAYER: see b200_hybrid_set_final_norm */
+  int32_t streams;                          /* HYPER layers: residual streams, 1 .. B200_MAX_STREAMS (0: other layouts) */
 } b200_hybrid_config;
 
 typedef struct b200_hybrid_layer {
@@ -947,7 +999,8 @@ typedef struct b200_hybrid_layer {
   const void* dist_slopes;                  /* fp32 [heads] or NULL */
   int32_t shared_cache;                     /* latent attention: != 0: no latent projection of its own; kv_cache is
                                                another (earlier) layer's cache, which this layer only reads */
-  int32_t expert_act, shared_act;           /* 0: SiLU(gate) * up ([gate | up] rows); 1: relu(up)^2 (up rows only) */
+  int32_t expert_act, shared_act;           /* 0: SiLU(gate) * up ([gate | up] rows); 1: relu(up)^2 (up rows only);
+                                               2 (shared_act): the exact GELU of up (up rows only) */
   int32_t identity_experts;                 /* router outputs experts .. experts + identity_experts - 1 return the input */
   int32_t route_groups, route_keep;         /* see b200_moe_route_ex (0: no groups) */
   int32_t shared_gated;                     /* != 0: one more row closes w_shared_gate_up; the shared expert's output is
@@ -957,7 +1010,7 @@ typedef struct b200_hybrid_layer {
    * attention, the delta rule with a decay per key channel, dense feed-forwards with biases */
   int32_t norm_kind;                        /* B200_NORM_* of norm_w (and ff_norm_w) */
   float norm_alpha, ff_norm_alpha;          /* DYNTANH: the scalar inside the tanh */
-  const void *norm_b, *ff_norm_b;           /* DYNTANH: fp32 [width] bias (NULL: none) */
+  const void *norm_b, *ff_norm_b;           /* DYNTANH, LAYER: fp32 [width] bias (NULL: none) */
   const void* shift_w;                      /* fp32 [width] or NULL: token shift of the mixer's input (b200_stream_norm) */
   void* shift_state;                        /* fp32 [slots, width], caller-owned */
   const void* depth_w;                      /* fp32 [layer + 2] or NULL: the layer's result X_(layer+1) is kept, and what
@@ -978,6 +1031,17 @@ typedef struct b200_hybrid_layer {
    * logits are w_gate2 low_g (w_gate2 fp32 [heads x vdim, gate_rank]) and the gate is a sigmoid (gate_act 1)          */
   int32_t chan_rank, gate_rank;
   const void* w_gate2;
+  /* ---- HYPER layers, learned distance bias, value mixing, sigmoid routers
+   * hc_*: connections of the mixer, ff_hc_*: of the feed-forward; fp32 in [streams], mix [streams, streams] (row: from,
+   * column: to), out [streams].                                                                                     */
+  const void *hc_in, *hc_mix, *hc_out, *ff_hc_in, *ff_hc_mix, *ff_hc_out;
+  const void* dist_bias;                    /* window attention: fp32 [heads, dist_n], see b200_attn_options */
+  int32_t dist_n;
+  int32_t v_mix_role;                       /* window attention: 1: this layer's values of a step are kept for later layers;
+                                               2: its values are mixed with them: (1 - v_mix) v + v_mix v_first.  All such
+                                               layers have the same kv_heads x vdim                                   */
+  float v_mix;
+  int32_t route_score, route_group_top, route_renorm;   /* see b200_moe_route_full (route_group_top 0 reads as 1) */
 } b200_hybrid_layer;
 
 typedef struct b200_hybrid b200_hybrid;
@@ -989,7 +1053,7 @@ void b200_hybrid_set_layer(b200_hybrid*, int32_t layer, const b200_hybrid_layer*
 void b200_hybrid_set_layer_side(b200_hybrid*, int32_t layer, const b200_hybrid_layer* side);
 /* embed [vocab, width], lm_head [vocab, width] in dtype dt; final_norm fp32 [width] */
 void b200_hybrid_set_globals(b200_hybrid*, const void* embed, const void* final_norm, const void* lm_head);
-/* final norm of kind DYNTANH: bias fp32 [width] (may be NULL) and the scalar inside the tanh */
+/* final norm of kind DYNTANH or LAYER: bias fp32 [width] (may be NULL) and the scalar inside the tanh */
 void b200_hybrid_set_final_norm(b200_hybrid*, const void* bias, float alpha);
 int64_t b200_hybrid_workspace_bytes(const b200_hybrid*);
 void b200_hybrid_set_workspace(b200_hybrid*, void* workspace, int64_t bytes);

@@ -52,7 +52,7 @@ class HybridConfig(C.Structure):
     _fields_ = [(n, c_i32) for n in ("width", "vocab", "num_layers", "dt", "block_size", "num_blocks",
                                      "max_blocks_per_seq", "max_seqs", "max_tokens", "num_state_slots")] + \
                [("norm_eps", c_f32), ("norm_weight_offset", c_f32), ("embed_scale", c_f32), ("embed_pos_base", c_f32),
-                ("final_norm_kind", c_i32)]
+                ("final_norm_kind", c_i32), ("streams", c_i32)]
 
 
 class AttnOptions(C.Structure):
@@ -60,7 +60,8 @@ class AttnOptions(C.Structure):
 
     _fields_ = [(n, c_i32) for n in ("head_norm", "v_from_k", "q_temp_every", "gate_elems")] + \
                [("q_temp_coef", c_f32), ("dist_slopes", c_vp), ("rot_half", c_i32), ("rot_mag", c_f32),
-                ("v_rot_freq", c_vp)] + [(n, c_i32) for n in ("v_heads", "chunk", "out_f32", "no_cache")]
+                ("v_rot_freq", c_vp)] + [(n, c_i32) for n in ("v_heads", "chunk", "out_f32", "no_cache")] + \
+               [("dist_bias", c_vp), ("dist_n", c_i32), ("v_mix", c_f32), ("v_first_out", c_vp), ("v_first", c_vp)]
 
 
 class HybridLayer(C.Structure):
@@ -88,7 +89,10 @@ class HybridLayer(C.Structure):
                [("ff_scale", c_f32), ("ff_up_bias", c_vp), ("ff_down_bias", c_vp)] + \
                [(n, c_i32) for n in ("rot_half", "chunk", "score_maps", "diff_norm")] + \
                [("diff_lambda", c_f32), ("diff_out_scale", c_f32), ("v_rot_freq", c_vp)] + \
-               [("chan_rank", c_i32), ("gate_rank", c_i32), ("w_gate2", c_vp)]
+               [("chan_rank", c_i32), ("gate_rank", c_i32), ("w_gate2", c_vp)] + \
+               [(n, c_vp) for n in ("hc_in", "hc_mix", "hc_out", "ff_hc_in", "ff_hc_mix", "ff_hc_out", "dist_bias")] + \
+               [("dist_n", c_i32), ("v_mix_role", c_i32), ("v_mix", c_f32)] + \
+               [(n, c_i32) for n in ("route_score", "route_group_top", "route_renorm")]
 
 
 class KvCachePlan(C.Structure):
@@ -280,6 +284,8 @@ _SIGS = {
     "b200_moe_route": (None, [c_vp, c_i32, c_i32, c_i32, c_f32, c_vp, c_vp, c_i64]),
     "b200_moe_workspace_bytes": (c_i64, [c_i32] * 5),
     "b200_moe_route_ex": (None, [c_vp, c_vp] + [c_i32] * 5 + [c_f32, c_vp, c_vp, c_i64]),
+    "b200_moe_route_full": (None, [c_vp, c_vp] + [c_i32] * 8 + [c_f32, c_vp, c_vp, c_i64]),
+    "b200_moe_experts_rows": (None, [c_vp] * 4 + [c_i32] * 7 + [c_vp, c_vp, c_vp, c_i64]),
     "b200_moe_experts_ex": (None, [c_vp] * 6 + [c_i32] * 8 + [c_vp, c_i32, c_i32, c_vp, c_i64]),
     "b200_moe_experts": (None, [c_vp] * 6 + [c_i32] * 6 + [c_vp, c_i64]),
     "b200_hybrid_new": (c_vp, [C.POINTER(HybridConfig)]),
@@ -290,6 +296,9 @@ _SIGS = {
     "b200_hybrid_set_final_norm": (None, [c_vp, c_vp, c_f32]),
     "b200_hybrid_workspace_bytes": (c_i64, [c_vp]),
     "b200_stream_norm": (None, [c_vp] * 4 + [c_f32, c_i32, c_f32, c_f32] + [c_vp] * 6 + [c_i32] * 4 + [c_i64]),
+    "b200_hyper_step": (None, [c_vp, c_vp, c_i64, c_vp, c_i64] + [c_vp] * 4 + [c_i32] + [c_vp] * 5 +
+                        [c_f32, c_i32, c_f32, c_f32, c_vp] + [c_i32] * 4 + [c_i64]),
+    "b200_ff_act": (None, [c_vp, c_vp, c_i32, c_vp] + [c_i32] * 4 + [c_i64]),
     "b200_depth_mix": (None, [c_vp, c_vp, c_i64, c_vp, c_i32, c_i64, c_i64]),
     "b200_attn_finish": (None, [c_vp, c_vp, c_vp, c_i32, c_i32, c_vp, c_vp, c_i32, c_i32, c_f32, c_i32, c_f32, c_f32,
                                 c_i32, c_i32, c_i32, c_i32, c_i64]),

@@ -32,6 +32,11 @@
 // h = ff_norm(x), x += ff_scale * ff(h).  With depth weights the layers' results X_0 (embedding) .. X_L are kept side by
 // side, layer i works in place on slot i + 1 (which starts as its input), and depth_mix writes
 // sum_j depth_w[j] X_j into slot i + 2 (the stream for the last layer), which is the next layer's input.
+// Hyper-connected layer (pre-norm sublayers over S residual streams): hyper_step = the update that closes the previous
+// sublayer (X_t <- sum_s mix[s][t] X_s + out[t] y), the next sublayer's weighted sum of the streams, its norm and the
+// rounding, in one pass; y = mixer(h); hyper_step; y = ff(h) -- routed experts leave their rows unsummed, the next
+// hyper_step weighs them.  The embedding row is written once and read as every stream by the first steps; the step behind
+// the last sublayer sums the streams of the wanted rows only and applies the final norm.
 //   window attention with rotated values, a chunked mask or two score maps: the attention writes fp32, attn_finish
 //                      combines the maps (a_0 - lambda a_1), turns rotated values back, norms per head, scales, gates
 //   delta rule, channel form: [q | k | v | b | low_a | low_g] = h W_in^T ; short_conv_silu ; lowrank_decay (kind 1)
@@ -74,6 +79,7 @@ struct b200_hybrid {
   // workspace carve-up
   float* x = nullptr;          // [T, width] residual stream
   float* y = nullptr;          // [T, width] output of a sublayer before the norm that follows it (sandwich layers)
+  float* vfirst = nullptr;     // [T, max kv_heads vdim] values of the step that later layers mix in (v_mix_role)
   void* h = nullptr;           // [T, width] normed stream, operand dtype
   const void* hin = nullptr;   // what the sublayers of the current layer read: h, or x itself (fp32 post-norm layers)
   float* proj = nullptr;       // [T, max fused input projection]
@@ -152,6 +158,7 @@ static int64_t carve(b200_hybrid* r, uint8_t* base) {
   const b200_hybrid_config& c = r->cfg;
   const size_t T = c.max_tokens, es = c.dt ? 4 : 2;
   size_t conv_n = 1, proj_n = 1, aux_n = 1, opa_n = 1, lat_n = 1, E = 1, top = 1, sh_n = 1, moe_bytes = 256, attn_bytes = 0;
+  size_t vfirst_n = 0;
   // rows up to which a step may split its attention rows: beyond two blocks per SM a split is never chosen
   r->attn_ws_rows = std::min<size_t>(T, 2 * static_cast<size_t>(sm_count()));
   std::vector<b200_hybrid_layer> all(r->layers);
@@ -163,6 +170,7 @@ static int64_t carve(b200_hybrid* r, uint8_t* base) {
       const int maps = l.score_maps > 1 ? l.score_maps : 1;
       aux_n = std::max<size_t>(aux_n, static_cast<size_t>(maps) * l.heads * l.dim);
       opa_n = std::max<size_t>(opa_n, static_cast<size_t>(l.heads) * l.vdim);
+      if (l.v_mix_role) vfirst_n = std::max<size_t>(vfirst_n, static_cast<size_t>(l.kv_heads) * l.vdim);
       if (needs_finish(l)) conv_n = std::max<size_t>(conv_n, static_cast<size_t>(maps) * l.heads * l.vdim);
       for (size_t rows = 1; rows <= r->attn_ws_rows; ++rows)
         attn_bytes = std::max(attn_bytes, window_attn_workspace_bytes(static_cast<int>(rows), maps * l.heads,
@@ -203,9 +211,10 @@ static int64_t carve(b200_hybrid* r, uint8_t* base) {
   };
   bool depth = false;
   for (const b200_hybrid_layer& l : r->layers) depth = depth || l.depth_w != nullptr;
-  r->x0 = r->x = (float*)take(T * c.width * 4);
+  r->x0 = r->x = (float*)take(static_cast<size_t>(std::max(c.streams, 1)) * T * c.width * 4);     // stream after stream
   r->hist = depth ? (float*)take((static_cast<size_t>(c.num_layers) + 1) * T * c.width * 4) : nullptr;
   r->y = (float*)take(T * c.width * 4);
+  r->vfirst = vfirst_n ? (float*)take(T * vfirst_n * 4) : nullptr;
   r->h = take(T * c.width * es);
   r->proj = (float*)take(T * proj_n * 4);
   r->conv = (float*)take(T * conv_n * 4);
@@ -238,7 +247,8 @@ extern "C" {
 
 b200_hybrid* b200_hybrid_new(const b200_hybrid_config* cfg) {
   if (!cfg || cfg->width <= 0 || cfg->vocab <= 0 || cfg->num_layers <= 0 || cfg->block_size != seqmix::kPage ||
-      cfg->max_seqs <= 0 || cfg->max_tokens <= 0 || (cfg->dt != 0 && cfg->dt != 1)) {
+      cfg->max_seqs <= 0 || cfg->max_tokens <= 0 || (cfg->dt != 0 && cfg->dt != 1) || cfg->streams < 0 ||
+      cfg->streams > B200_MAX_STREAMS) {
     set_error(1, "hybrid_new: bad config");
     return nullptr;
   }
@@ -265,7 +275,8 @@ static bool mixer_ok(const b200_hybrid_layer* l) {
            l->rot_dims <= l->dim && (l->rot_dims == 0 || l->rot_freq) && l->kv_cache && l->v_cache &&
            (!l->v_from_k || l->vdim == l->dim) && l->gated >= 0 && l->gated <= 2 && l->score_maps >= 0 &&
            l->score_maps <= 2 && (l->score_maps < 2 || (!l->v_from_k && !l->sink)) && l->chunk >= 0 &&
-           (!l->v_rot_freq || (l->vdim % 2 == 0 && !l->v_from_k));
+           (!l->v_rot_freq || (l->vdim % 2 == 0 && !l->v_from_k)) && (!l->dist_bias || l->dist_n > 0) &&
+           l->v_mix_role >= 0 && l->v_mix_role <= 2 && (l->v_mix_role == 0 || !l->shared_cache);
   if (l->mixer == B200_MIXER_DECAY_ATTN)
     return ok && l->dim > 0 && l->dim <= 256 && l->rec_state && l->norm_groups > 0 &&
            (l->heads * l->vdim) % l->norm_groups == 0 && (l->out_norm_period == 0 || l->out_norm_w) &&
@@ -295,13 +306,19 @@ void b200_hybrid_set_layer(b200_hybrid* r, int32_t layer, const b200_hybrid_laye
   else if (l->layout == B200_LAYOUT_POSTNORM)
     ok = ok && l->post_norm_w && ((l->shared_ff == 0 && l->experts == 0) || l->ff_post_norm_w);
   else
-    ok = ok && l->norm_w && (l->layout == B200_LAYOUT_PARALLEL || l->layout == B200_LAYOUT_PRENORM);
+    ok = ok && l->norm_w &&
+         (l->layout == B200_LAYOUT_PARALLEL || l->layout == B200_LAYOUT_PRENORM || l->layout == B200_LAYOUT_HYPER);
+  const bool hyper = l->layout == B200_LAYOUT_HYPER, with_ff = l->shared_ff > 0 || l->experts > 0;
+  ok = ok && hyper == (r->cfg.streams > 0);
+  if (hyper)
+    ok = ok && l->hc_in && l->hc_mix && l->hc_out && !l->shift_w && !l->depth_w && l->out_scale == 1.f && l->ff_scale == 1.f &&
+         (!with_ff || (l->ff_norm_w && l->ff_hc_in && l->ff_hc_mix && l->ff_hc_out));
   if (l->layout == B200_LAYOUT_PRENORM)
     ok = ok && ((l->shared_ff == 0 && l->experts == 0) || l->ff_norm_w) && (l->experts == 0 || l->ff_scale == 1.f);
-  ok = ok && (l->norm_kind == B200_NORM_RMS || l->norm_kind == B200_NORM_DYNTANH) && (!l->shift_w || l->shift_state) &&
+  ok = ok && l->norm_kind >= B200_NORM_RMS && l->norm_kind <= B200_NORM_LAYER && (!l->shift_w || l->shift_state) &&
        ((!l->shift_w && !l->depth_w && !l->ff_up_bias && !l->ff_down_bias && l->norm_kind == B200_NORM_RMS) ||
-        l->layout == B200_LAYOUT_PRENORM) &&
-       ((!l->ff_up_bias && !l->ff_down_bias) || (l->shared_ff > 0 && l->shared_act == 1 && !l->shared_gated));
+        l->layout == B200_LAYOUT_PRENORM || hyper) &&
+       ((!l->ff_up_bias && !l->ff_down_bias) || (l->shared_ff > 0 && l->shared_act != 0 && !l->shared_gated));
   if (l->mixer == B200_MIXER_WINDOW_ATTN || l->mixer == B200_MIXER_DECAY_ATTN)
     ok = ok && mixer_ok(l);
   else if (l->mixer == B200_MIXER_LATENT_ATTN)
@@ -322,13 +339,14 @@ void b200_hybrid_set_layer(b200_hybrid* r, int32_t layer, const b200_hybrid_laye
     const int all = l->experts + l->identity_experts;
     ok = ok && l->identity_experts >= 0 && l->top > 0 && l->top <= all && l->expert_ff > 0 && l->w_router &&
          l->w_gate_up && l->w_down && (l->expert_act == 0 || l->expert_act == 1) && l->route_groups >= 0 &&
+         (l->route_score == 0 || l->route_score == 1) && l->route_group_top >= 0 && l->route_group_top <= 2 &&
          (l->route_groups == 0 || (all % l->route_groups == 0 && l->route_keep >= 1 && l->route_keep <= l->route_groups &&
                                    l->top <= all / l->route_groups * l->route_keep));
   } else {
     ok = ok && l->identity_experts == 0;
   }
   if (l->shared_ff > 0)
-    ok = ok && l->w_shared_gate_up && l->w_shared_down && (l->shared_act == 0 || l->shared_act == 1) &&
+    ok = ok && l->w_shared_gate_up && l->w_shared_down && l->shared_act >= 0 && l->shared_act <= 2 &&
          (!l->shared_gated || l->shared_act == 1);
   if (!ok) {
     set_error(1, "hybrid_set_layer: inconsistent layer description");
@@ -512,6 +530,11 @@ static void mixer_window(b200_hybrid* r, const b200_hybrid_layer& l, const int64
   opt.chunk = l.chunk;
   opt.out_f32 = finish;
   opt.no_cache = l.shared_cache;
+  opt.dist_bias = (const float*)l.dist_bias;
+  opt.dist_n = l.dist_n;
+  opt.v_mix = l.v_mix;
+  opt.v_first_out = l.v_mix_role == 1 ? r->vfirst : nullptr;
+  opt.v_first = l.v_mix_role == 2 ? r->vfirst : nullptr;
   launch_window_attn_prep(r->proj, n_in, (const float*)l.in_bias, (const float*)l.q_norm_w, (const float*)l.k_norm_w,
                           l.rot_freq, positions, slots, r->aux, l.kv_cache, l.v_cache, T, maps * H, maps * G, l.dim,
                           l.vdim, l.rot_dims, c.norm_eps, c.dt, &opt, st);
@@ -582,6 +605,15 @@ static void dense_ffn(b200_hybrid* r, const b200_hybrid_layer& l, int T, cudaStr
               0, c.dt, st);
 }
 
+// the router of a layer: logits, choice and weights of every token
+static void route_tokens(b200_hybrid* r, const b200_hybrid_layer& l, int T, cudaStream_t st) {
+  const b200_hybrid_config& c = r->cfg;
+  const int all = l.experts + l.identity_experts;
+  gemm_f32out(r->hin, c.width, 0, l.w_router, c.width, 0, r->rlog, all, 0, T, all, c.width, 1, 0.f, 0, c.dt, st);
+  launch_moe_route(r->rlog, (const float*)l.route_bias, T, all, l.top, l.route_groups, l.route_keep, l.route_score,
+                   l.route_group_top, l.route_renorm, l.route_scale, r->top_idx, r->top_w, st);
+}
+
 // routed experts and their shared expert: dst = (accumulate ? dst : 0) + experts(h) + shared(h).  `ident` / `ident_f32`:
 // the rows that identity experts return (the sublayer's input before any rounding, where the layer has it in fp32).
 // `scale` multiplies the shared / dense part (routed experts take none).
@@ -589,24 +621,21 @@ static void feed_forward(b200_hybrid* r, const b200_hybrid_layer& l, int T, floa
                          int ident_f32, cudaStream_t st, float scale = 1.f) {
   const b200_hybrid_config& c = r->cfg;
   if (l.experts > 0) {
-    const int all = l.experts + l.identity_experts;
-    gemm_f32out(r->hin, c.width, 0, l.w_router, c.width, 0, r->rlog, all, 0, T, all, c.width, 1, 0.f, 0, c.dt, st);
-    launch_moe_route(r->rlog, (const float*)l.route_bias, T, all, l.top, l.route_groups, l.route_keep, l.route_scale,
-                     r->top_idx, r->top_w, st);
+    route_tokens(r, l, T, st);
     b200_moe_experts_ex(dst, r->hin, r->top_idx, r->top_w, l.w_gate_up, l.w_down, T, l.experts, l.identity_experts, l.top,
                         c.width, l.expert_ff, l.expert_act, accumulate ? 1 : 0, ident, ident_f32, c.dt, r->moe_ws,
                         reinterpret_cast<int64_t>(st));
     accumulate = true;
   }
   if (l.shared_ff > 0) {
-    // SiLU-gated: [gate | up] rows; squared ReLU: up rows, closed by the one row of the token's gate where there is one
+    // SiLU-gated: [gate | up] rows; squared ReLU, GELU: up rows, closed by the one row of the token's gate where there is one
     const int rows = l.shared_act == 0 ? 2 * l.shared_ff : l.shared_ff + (l.shared_gated ? 1 : 0);
     gemm_f32out(r->hin, c.width, 0, l.w_shared_gate_up, c.width, 0, r->sh, rows, 0, T, rows, c.width, 1, 0.f, 0, c.dt, st);
     if (l.shared_act == 0)
       launch_silu_mul_f32(r->sha, r->sh, T, l.shared_ff, c.dt, st);
     else
-      launch_relu2_f32(r->sha, r->sh, rows, T, l.shared_ff, l.shared_gated ? l.shared_ff : -1,
-                       (const float*)l.ff_up_bias, c.dt, st);
+      launch_ff_act(r->sha, r->sh, rows, T, l.shared_ff, l.shared_gated ? l.shared_ff : -1, (const float*)l.ff_up_bias,
+                    l.shared_act, c.dt, st);
     gemm_f32out_scaled(r->sha, l.shared_ff, 0, l.w_shared_down, l.shared_ff, 0, dst, c.width, 0, T, c.width, l.shared_ff,
                        1, scale, accumulate ? 1.f : 0.f, 0, c.dt, st);
     if (l.ff_down_bias) launch_bias_rows(dst, (const float*)l.ff_down_bias, scale, T, c.width, st);
@@ -640,6 +669,25 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
     r->x = r->hist + hstride;
   }
   bool h_is_x = first_reads_stream;          // h holds the bf16 rounding of the current x
+  // hyper-connected streams: the update of the sublayer run last waits for the next read of the streams, which does both
+  struct {
+    const float *mix = nullptr, *out = nullptr, *y = nullptr, *down = nullptr;
+    const int32_t* slot_of_pair = nullptr;
+    int top = 0;
+  } pend;
+  size_t sstride = 0;                        // between the streams as they lie now; 0: all equal the embedding rows
+  const size_t sfull = static_cast<size_t>(c.max_tokens) * c.width;
+  auto hyper = [&](void* out, bool store, const float* in_w, const float* w, const float* b, float alpha, int kind,
+                   const uint32_t* rows, int n) {
+    const bool update = pend.mix != nullptr;
+    launch_hyper_step(out, update && store ? r->x : nullptr, sfull, r->x, sstride, pend.y, pend.down, pend.slot_of_pair,
+                      r->top_w, pend.top, pend.mix, pend.out, in_w, w, b, alpha, kind, c.norm_eps, c.norm_weight_offset, rows,
+                      c.streams, n, c.width, c.dt, st);
+    if (update && store) {
+      sstride = sfull;
+      pend = {};
+    }
+  };
   for (int i = 0; i < c.num_layers; ++i) {
     const b200_hybrid_layer& l = r->layers[i];
     const b200_hybrid_layer& side = r->sides[i];
@@ -673,6 +721,36 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
       continue;
     }
     h_is_x = false;
+    if (l.layout == B200_LAYOUT_HYPER) {
+      hyper(r->h, true, (const float*)l.hc_in, (const float*)l.norm_w, (const float*)l.norm_b, l.norm_alpha, l.norm_kind,
+            nullptr, T);
+      run_mixer(r, l, positions, slot_mapping, cu, ctx, block_tables, state_slots, max_blocks, B, T, r->y, l.out_scale,
+                0.f, st);
+      if (side.heads > 0)
+        run_mixer(r, side, positions, slot_mapping, cu, ctx, block_tables, state_slots, max_blocks, B, T, r->y,
+                  side.out_scale, 1.f, st);
+      pend = {(const float*)l.hc_mix, (const float*)l.hc_out, r->y, nullptr, nullptr, 0};
+      if (l.experts > 0 || l.shared_ff > 0) {
+        hyper(r->h, true, (const float*)l.ff_hc_in, (const float*)l.ff_norm_w, (const float*)l.ff_norm_b, l.ff_norm_alpha,
+              l.norm_kind, nullptr, T);
+        pend = {(const float*)l.ff_hc_mix, (const float*)l.ff_hc_out, r->y, nullptr, nullptr, 0};
+        if (l.experts > 0 && l.shared_ff == 0 && l.identity_experts == 0) {      // the next hyper_step sums the experts' rows
+          route_tokens(r, l, T, st);
+          b200_moe_experts_rows(r->hin, r->top_idx, l.w_gate_up, l.w_down, T, l.experts, l.top, c.width, l.expert_ff,
+                                l.expert_act, c.dt, r->moe_ws, &pend.down, &pend.slot_of_pair, stream);
+          pend.y = nullptr;
+          pend.top = l.top;
+        } else {
+          feed_forward(r, l, T, r->y, false, r->h, 0, st);
+        }
+      }
+      if (r->trace) {                        // the sum of the streams after the layer
+        hyper(nullptr, true, nullptr, nullptr, nullptr, 1.f, l.norm_kind, nullptr, T);
+        launch_depth_mix(r->trace + static_cast<size_t>(i) * sfull, r->x, sstride, nullptr, c.streams,
+                         static_cast<size_t>(T) * c.width, st);
+      }
+      continue;
+    }
     if (l.layout == B200_LAYOUT_PRENORM) {
       launch_stream_norm(r->h, r->x, (const float*)l.norm_w, (const float*)l.norm_b, l.norm_alpha, l.norm_kind, c.norm_eps,
                          c.norm_weight_offset, nullptr, (const float*)l.shift_w, (float*)l.shift_state, state_slots, cu,
@@ -730,7 +808,10 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
                       static_cast<size_t>(T) * c.width * 4, cudaMemcpyDeviceToDevice, st);
   }
   if (num_out > 0) {
-    if (c.final_norm_kind == B200_NORM_RMS)
+    if (c.streams > 0)
+      hyper(r->hr, false, nullptr, (const float*)r->final_norm, (const float*)r->final_norm_b, r->final_norm_alpha,
+            c.final_norm_kind, out_rows, num_out);
+    else if (c.final_norm_kind == B200_NORM_RMS)
       launch_resid_rmsnorm(r->hr, r->x, (const float*)r->final_norm, num_out, c.width, c.norm_eps, c.norm_weight_offset,
                            out_rows, c.dt, st);
     else

@@ -5,7 +5,9 @@
 //   route    : s = softmax(logits) over all experts (fp32); the `top` largest choice scores (ties: lowest index) keep
 //              their own probability times `scale`; nothing is renormalised.  The choice score is s plus an optional
 //              per-expert bias; with groups, the experts form equal runs of neighbours, a run's score is its largest
-//              choice score, and members of all but the `keep` best runs cannot be chosen.
+//              choice score (or the sum of its two largest), and members of all but the `keep` best runs cannot be
+//              chosen.  Options: s = sigmoid(logit) per expert instead of the softmax; the chosen weights divided by
+//              their sum.
 //   sort     : pair p = token * top + choice; pairs are bucketed by expert into slots [off[e], off[e+1]).  The order
 //              inside a bucket is arbitrary and does not influence any result: every pair is one independent row.
 //   gate_up  : act[slot, f] = silu(h[token] . Wg[e, f]) * (h[token] . Wu[e, f]);  W_gate_up [E, 2F, width] (gate rows
@@ -24,8 +26,8 @@ using namespace seqmix;
 
 // one warp per token.  sm per warp: s[E] (probabilities) | c[E] (choice scores; -inf: not available) | gs[groups]
 __global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int E, int top,
-                                 int groups, int keep, float scale, int32_t* __restrict__ top_idx,
-                                 float* __restrict__ top_w) {
+                                 int groups, int keep, int score, int group_top, int renorm, float scale,
+                                 int32_t* __restrict__ top_idx, float* __restrict__ top_w) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int t = blockIdx.x * nw + warp;
@@ -34,29 +36,40 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
   float* c = s + E;
   float* gs = c + E;
   const float* z = logits + static_cast<size_t>(t) * E;
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-  mx = lanes_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float p = expf(z[e] - mx);
-    s[e] = p;
-    sum += p;
-  }
-  sum = lanes_sum(sum);
-  __syncwarp();
-  for (int e = lane; e < E; e += 32) {
-    const float p = s[e] / sum;
-    s[e] = p;
-    c[e] = p + (bias ? bias[e] : 0.f);
+  if (score == 0) {
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = lanes_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(z[e] - mx);
+      s[e] = p;
+      sum += p;
+    }
+    sum = lanes_sum(sum);
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) {
+      const float p = s[e] / sum;
+      s[e] = p;
+      c[e] = p + (bias ? bias[e] : 0.f);
+    }
+  } else {
+    for (int e = lane; e < E; e += 32) {
+      const float p = sigmoid_f(z[e]);
+      s[e] = p;
+      c[e] = p + (bias ? bias[e] : 0.f);
+    }
   }
   __syncwarp();
   if (groups > 0) {
     const int per = E / groups;
     for (int g = lane; g < groups; g += 32) {
-      float best = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, c[e]);
-      gs[g] = best;
+      float best = -INFINITY, second = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        second = fmaxf(second, fminf(best, c[e]));
+        best = fmaxf(best, c[e]);
+      }
+      gs[g] = best + (group_top == 2 && per > 1 ? second : 0.f);
     }
     __syncwarp();
     // a run stays available while fewer than `keep` runs beat it (a tie goes to the lower index)
@@ -68,6 +81,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
     }
     __syncwarp();
   }
+  float total = 0.f;             // sum of the chosen scores
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
     int bi = E;
@@ -87,14 +101,17 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
         bi = oi;
       }
     }
+    if (bi >= E) bi = 0;       // fewer available experts than `top` (rejected by the launcher; keeps the index valid)
+    total += s[bi];
     if (lane == 0) {
-      if (bi >= E) bi = 0;     // fewer available experts than `top` (rejected by the launcher; keeps the index valid)
       top_idx[static_cast<size_t>(t) * top + j] = bi;
       top_w[static_cast<size_t>(t) * top + j] = s[bi] * scale;
       c[bi] = -INFINITY;
     }
     __syncwarp();
   }
+  if (renorm)
+    for (int j = lane; j < top; j += 32) top_w[static_cast<size_t>(t) * top + j] /= total + 1e-20f;
 }
 
 // single block: histogram, exclusive scan, scatter
@@ -362,9 +379,14 @@ __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restric
   }
 }
 
-void launch_moe_route(const float* logits, const float* bias, int T, int E, int top, int groups, int keep, float scale,
-                      int32_t* top_idx, float* top_w, cudaStream_t st_) {
+void launch_moe_route(const float* logits, const float* bias, int T, int E, int top, int groups, int keep, int score,
+                      int group_top, int renorm, float scale, int32_t* top_idx, float* top_w, cudaStream_t st_) {
   if (T <= 0) return;
+  if (group_top == 0) group_top = 1;
+  if (score < 0 || score > 1 || group_top < 1 || group_top > 2) {
+    set_error(1, "moe_route: unknown score, or a group score of more than two members");
+    return;
+  }
   if (groups < 0 || (groups > 0 && (E % groups != 0 || keep < 1 || keep > groups))) {
     set_error(1, "moe_route: the experts do not split into that many equal groups, or keep is out of range");
     return;
@@ -377,8 +399,8 @@ void launch_moe_route(const float* logits, const float* bias, int T, int E, int 
     set_error(1, "moe_route: too many experts, or top above the number that can be chosen");
     return;
   }
-  moe_route_kernel<<<(T + nw - 1) / nw, nw * 32, nw * per_warp, st_>>>(logits, bias, T, E, top, groups, keep, scale,
-                                                                      top_idx, top_w);
+  moe_route_kernel<<<(T + nw - 1) / nw, nw * 32, nw * per_warp, st_>>>(logits, bias, T, E, top, groups, keep, score,
+                                                                      group_top, renorm, scale, top_idx, top_w);
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -453,14 +475,21 @@ extern "C" {
 void b200_moe_route(const float* logits, int32_t num_tokens, int32_t experts, int32_t top, float scale,
                     int32_t* top_idx, float* top_w, int64_t stream) {
   B200_CHECK_ARG(logits && top_idx && top_w && experts > 0 && top > 0, "moe_route: bad arguments");
-  b200::launch_moe_route(logits, nullptr, num_tokens, experts, top, 0, 0, scale, top_idx, top_w,
+  b200::launch_moe_route(logits, nullptr, num_tokens, experts, top, 0, 0, 0, 1, 0, scale, top_idx, top_w,
                          reinterpret_cast<cudaStream_t>(stream));
 }
 void b200_moe_route_ex(const float* logits, const float* bias, int32_t num_tokens, int32_t experts, int32_t top,
                        int32_t groups, int32_t keep, float scale, int32_t* top_idx, float* top_w, int64_t stream) {
   B200_CHECK_ARG(logits && top_idx && top_w && experts > 0 && top > 0, "moe_route_ex: bad arguments");
-  b200::launch_moe_route(logits, bias, num_tokens, experts, top, groups, keep, scale, top_idx, top_w,
+  b200::launch_moe_route(logits, bias, num_tokens, experts, top, groups, keep, 0, 1, 0, scale, top_idx, top_w,
                          reinterpret_cast<cudaStream_t>(stream));
+}
+void b200_moe_route_full(const float* logits, const float* bias, int32_t num_tokens, int32_t experts, int32_t top,
+                         int32_t groups, int32_t keep, int32_t score, int32_t group_top, int32_t renorm, float scale,
+                         int32_t* top_idx, float* top_w, int64_t stream) {
+  B200_CHECK_ARG(logits && top_idx && top_w && experts > 0 && top > 0, "moe_route_full: bad arguments");
+  b200::launch_moe_route(logits, bias, num_tokens, experts, top, groups, keep, score, group_top, renorm, scale, top_idx,
+                         top_w, reinterpret_cast<cudaStream_t>(stream));
 }
 // The experts' feed-forward of routed tokens, added into the fp32 stream x [T, width]: h [T, width] and the weights
 // in the activation dtype (dt 0 bf16, 1 fp32).  workspace: b200_moe_workspace_bytes() bytes.
@@ -468,15 +497,14 @@ int64_t b200_moe_workspace_bytes(int32_t num_tokens, int32_t experts, int32_t to
   const int64_t P = static_cast<int64_t>(num_tokens) * top;
   return 256 * 6 + (experts + 1) * 4 + P * 8 + P * ff * 4 + P * width * 4;
 }
-void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, const float* top_w, const void* w_up,
-                         const void* w_down, int32_t num_tokens, int32_t experts, int32_t identity, int32_t top,
-                         int32_t width, int32_t ff, int32_t act, int32_t accumulate, const void* ident,
-                         int32_t ident_f32, int32_t dt, void* workspace, int64_t stream) {
-  B200_CHECK_ARG(out && h && top_idx && top_w && w_up && w_down && workspace && (dt == 0 || dt == 1) &&
-                     (act == 0 || act == 1) && identity >= 0 && (identity == 0 || ident),
-                 "moe_experts: bad arguments");
-  cudaStream_t st_ = reinterpret_cast<cudaStream_t>(stream);
-  const int P = num_tokens * top, all = experts + identity;
+}
+
+namespace b200 {
+// buckets, both grouped products; the rows of the (token, choice) pairs and their places stay in the workspace
+static void moe_expert_rows(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down, int T, int experts,
+                            int identity, int top, int width, int ff, int act, int dt, void* workspace,
+                            const float** down_out, const int32_t** slot_out, cudaStream_t st_) {
+  const int P = T * top, all = experts + identity;
   auto up = [](size_t v) { return (v + 255) / 256 * 256; };
   uint8_t* p = reinterpret_cast<uint8_t*>(up(reinterpret_cast<size_t>(workspace)));
   int32_t* off = reinterpret_cast<int32_t*>(p); p += up((all + 1) * 4);
@@ -485,11 +513,39 @@ void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, cons
   void* actb = p; p += up(static_cast<size_t>(P) * ff * 4);
   float* down = reinterpret_cast<float*>(p);
   // identity experts take buckets past the real ones; the grouped products walk the first `experts` buckets only
-  b200::launch_moe_sort(top_idx, P, all, off, pos, sop, st_);
-  b200::launch_moe_gate_up(actb, h, w_up, off, pos, P, top, experts, width, ff, act, dt, st_);
-  b200::launch_moe_down(down, actb, w_down, off, P, experts, width, ff, dt, st_);
+  launch_moe_sort(top_idx, P, all, off, pos, sop, st_);
+  launch_moe_gate_up(actb, h, w_up, off, pos, P, top, experts, width, ff, act, dt, st_);
+  launch_moe_down(down, actb, w_down, off, P, experts, width, ff, dt, st_);
+  *down_out = down;
+  *slot_out = sop;
+}
+}  // namespace b200
+
+extern "C" {
+void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, const float* top_w, const void* w_up,
+                         const void* w_down, int32_t num_tokens, int32_t experts, int32_t identity, int32_t top,
+                         int32_t width, int32_t ff, int32_t act, int32_t accumulate, const void* ident,
+                         int32_t ident_f32, int32_t dt, void* workspace, int64_t stream) {
+  B200_CHECK_ARG(out && h && top_idx && top_w && w_up && w_down && workspace && (dt == 0 || dt == 1) &&
+                     (act == 0 || act == 1) && identity >= 0 && (identity == 0 || ident),
+                 "moe_experts: bad arguments");
+  cudaStream_t st_ = reinterpret_cast<cudaStream_t>(stream);
+  const float* down = nullptr;
+  const int32_t* sop = nullptr;
+  b200::moe_expert_rows(h, top_idx, w_up, w_down, num_tokens, experts, identity, top, width, ff, act, dt, workspace, &down,
+                        &sop, st_);
   b200::launch_moe_combine(out, down, sop, top_idx, top_w, num_tokens, top, width, experts, identity ? ident : nullptr,
                            ident_f32, dt, accumulate, st_);
+}
+void b200_moe_experts_rows(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down,
+                           int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff, int32_t act,
+                           int32_t dt, void* workspace, const float** down, const int32_t** slot_of_pair,
+                           int64_t stream) {
+  B200_CHECK_ARG(h && top_idx && w_up && w_down && workspace && down && slot_of_pair && (dt == 0 || dt == 1) &&
+                     (act == 0 || act == 1),
+                 "moe_experts_rows: bad arguments");
+  b200::moe_expert_rows(h, top_idx, w_up, w_down, num_tokens, experts, 0, top, width, ff, act, dt, workspace, down,
+                        slot_of_pair, reinterpret_cast<cudaStream_t>(stream));
 }
 void b200_moe_experts(float* x, const void* h, const int32_t* top_idx, const float* top_w, const void* w_gate_up,
                       const void* w_down, int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff,

@@ -2,7 +2,8 @@
 // stream (weight stored either plainly or as an offset from one), the grouped RMS norm with a SiLU gate that follows
 // a recurrent mixer (gate applied before or after the normalisation), SiLU * mul over an fp32 gate|up block, and
 // the rounding of fp32 rows to the dtype that feeds the next matrix product, the norm of the stream with a choice of
-// kind (RMS / dynamic tanh) and a token shift, and the weighted sum of the stored results of earlier layers.  All arithmetic is fp32; the output
+// kind (RMS / dynamic tanh / layer norm) and a token shift, the weighted sum of the stored results of earlier layers, and
+// the step between two sublayers of hyper-connected streams (update, read, norm).  All arithmetic is fp32; the output
 // dtype is bf16 or fp32.  Beside the fp16 / bf16 row kernels of glue.cu (rmsnorm_kernel, silu_mul_kernel), which
 // keep a 16-bit residual.
 #include "../../include/b200_vllm.h"
@@ -121,20 +122,26 @@ __global__ void silu_mul_f32_kernel(T* __restrict__ out, const float* __restrict
   }
 }
 
-template <typename T>
-__global__ void relu2_f32_kernel(T* __restrict__ out, const float* __restrict__ up, int ld, int ff, int gate_col,
-                                 const float* __restrict__ bias, size_t total) {
+// out[t, d] = act(up[t, d] + bias[d]) (* sigmoid(up[t, gate_col]) when gate_col >= 0); ACT 1: relu(.)^2, 2: the exact GELU
+template <typename T, int ACT>
+__global__ void ff_act_kernel(T* __restrict__ out, const float* __restrict__ up, int ld, int ff, int gate_col,
+                              const float* __restrict__ bias, size_t total) {
   for (size_t i = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; i < total;
        i += static_cast<size_t>(gridDim.x) * blockDim.x) {
     const size_t t = i / ff, d = i % ff;
-    const float u = fmaxf(up[t * ld + d] + (bias ? bias[d] : 0.f), 0.f);
+    const float z = up[t * ld + d] + (bias ? bias[d] : 0.f);
     const float g = gate_col >= 0 ? sigmoid_f(up[t * ld + gate_col]) : 1.f;
-    st(out + i, u * u * g);
+    if (ACT == 1) {
+      const float u = fmaxf(z, 0.f);
+      st(out + i, u * u * g);
+    } else {
+      st(out + i, 0.5f * z * (1.f + erff(z * 0.70710678118654752f)) * g);
+    }
   }
 }
 
-// One block per output row: a norm of the stream (RMS, or the dynamic tanh  tanh(alpha x) w + b  that needs no
-// statistics) and, with shift_w, the token shift behind it:  out[t] = n[t] + (n[t-1] - n[t]) * shift_w, where n[t-1] is
+// One block per output row: a norm of the stream (RMS, layer norm, or the dynamic tanh  tanh(alpha x) w + b  that needs
+// no statistics) and, with shift_w, the token shift behind it:  out[t] = n[t] + (n[t-1] - n[t]) * shift_w, where n[t-1] is
 // the un-shifted norm of the sequence's previous token -- recomputed from the row above, or, for the first row of a
 // portion, read from the sequence's shift state (zeros at position 0).  The block of a sequence's FIRST row also writes
 // the state: the un-shifted norm of the sequence's last row of the step.  Every thread reads the state entries it later
@@ -149,18 +156,23 @@ __global__ void stream_norm_kernel(T* __restrict__ out, const float* __restrict_
   const int r = blockIdx.x;
   const int t = rows ? static_cast<int>(rows[r]) : r;
   const float* xr = x + static_cast<size_t>(t) * width;
-  // inverse root mean square of a row (RMS kind only)
-  auto inv_rms = [&](const float* row) {
-    float ss = 0.f;
-    for (int d = threadIdx.x; d < width; d += blockDim.x) ss += row[d] * row[d];
+  // (mean, inverse root mean square of what is left of the mean) of a row; the RMS kind has no mean
+  auto stats = [&](const float* row) {
+    float mean = 0.f, ss = 0.f;
+    if (kind == B200_NORM_LAYER) {
+      for (int d = threadIdx.x; d < width; d += blockDim.x) mean += row[d];
+      mean = block_sum(mean, red) / static_cast<float>(width);
+    }
+    for (int d = threadIdx.x; d < width; d += blockDim.x) ss += (row[d] - mean) * (row[d] - mean);
     ss = block_sum(ss, red);
-    return 1.f / sqrtf(ss / static_cast<float>(width) + eps);
+    return make_float2(mean, 1.f / sqrtf(ss / static_cast<float>(width) + eps));
   };
-  auto normed = [&](const float* row, float inv, int d) {
-    return kind == B200_NORM_DYNTANH ? tanhf(alpha * row[d]) * w[d] + (bias ? bias[d] : 0.f)
-                                     : row[d] * inv * (w_offset + w[d]);
+  auto normed = [&](const float* row, float2 m, int d) {
+    const float b = bias ? bias[d] : 0.f;
+    return kind == B200_NORM_DYNTANH ? tanhf(alpha * row[d]) * w[d] + b : (row[d] - m.x) * m.y * (w_offset + w[d]) + b;
   };
-  const float inv = kind == B200_NORM_DYNTANH ? 1.f : inv_rms(xr);
+  const float2 none = make_float2(0.f, 1.f);
+  const float2 inv = kind == B200_NORM_DYNTANH ? none : stats(xr);
   if (!shift_w) {
     for (int d = threadIdx.x; d < width; d += blockDim.x) st(out + static_cast<size_t>(r) * width + d, normed(xr, inv, d));
     return;
@@ -172,8 +184,8 @@ __global__ void stream_norm_kernel(T* __restrict__ out, const float* __restrict_
   float* sp = shift_state + static_cast<size_t>(slots[b]) * width;
   const float* xp = xr - width;                                      // the row above (same sequence unless `first`)
   const float* xl = x + static_cast<size_t>(t1 - 1) * width;         // the sequence's last row of the step
-  const float inv_p = (kind == B200_NORM_DYNTANH || first) ? 1.f : inv_rms(xp);
-  const float inv_l = (kind == B200_NORM_DYNTANH || !first) ? 1.f : (t1 - 1 == t ? inv : inv_rms(xl));
+  const float2 inv_p = (kind == B200_NORM_DYNTANH || first) ? none : stats(xp);
+  const float2 inv_l = (kind == B200_NORM_DYNTANH || !first) ? none : (t1 - 1 == t ? inv : stats(xl));
   for (int d = threadIdx.x; d < width; d += blockDim.x) {
     const float n = normed(xr, inv, d);
     const float prev = first ? (fresh ? 0.f : sp[d]) : normed(xp, inv_p, d);
@@ -182,7 +194,155 @@ __global__ void stream_norm_kernel(T* __restrict__ out, const float* __restrict_
   }
 }
 
-// out[i] = sum_j w[j] * hist[j * stride + i], V floats per thread and step
+// One block per row: the step between two sublayers of hyper-connected streams (see b200_hyper_step).  A thread owns the
+// same columns in every stream, so the streams can be rewritten in place: it reads a column of all S old streams and of
+// the sublayer's row, forms every new stream from them, stores it, and keeps only the next sublayer's weighted sum, which
+// the block then norms from shared memory (mean first, then the squared deviations from it).  The S x S matrix and the
+// weight vectors sit in shared memory.
+struct HyperArgs {
+  void* out;
+  float* x_out;
+  size_t out_stride;
+  const float* x_in;
+  size_t in_stride;
+  const float *y, *down;
+  const int32_t* slot_of_pair;
+  const float* top_w;
+  int top;
+  const float *mix, *out_w, *in_w, *w, *bias;
+  float alpha;
+  int kind;
+  float eps, w_offset;
+  const uint32_t* rows;
+  int streams, width;
+};
+template <int V> struct FloatVec;
+template <> struct FloatVec<1> {
+  float v[1];
+  __device__ __forceinline__ void load(const float* p) { v[0] = *p; }
+  __device__ __forceinline__ void store(float* p) const { *p = v[0]; }
+};
+template <> struct FloatVec<4> {
+  float v[4];
+  __device__ __forceinline__ void load(const float* p) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+  }
+  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+};
+template <int V> __device__ __forceinline__ void store_vec(float* p, const FloatVec<V>& f) { f.store(p); }
+template <int V> __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const FloatVec<V>& f) {
+  if constexpr (V == 4) {
+    __nv_bfloat162 q[2] = {__floats2bfloat162_rn(f.v[0], f.v[1]), __floats2bfloat162_rn(f.v[2], f.v[3])};
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(q);
+  } else {
+    *p = __float2bfloat16_rn(f.v[0]);
+  }
+}
+template <typename T, int MS, int V>
+__global__ void hyper_step_kernel(const HyperArgs a) {
+  // red[36] | mix[S * S] | out_w[S] | in_w[S] | choice weights[top] | choice rows[top] | u[width] (16-byte aligned)
+  extern __shared__ __align__(16) float sm[];
+  const int S = a.streams, r = blockIdx.x, width = a.width;
+  float* red = sm;
+  float* mix = red + 36;
+  float* ow = mix + S * S;
+  float* iw = ow + S;
+  float* cw = iw + S;
+  int* cr = reinterpret_cast<int*>(cw + a.top);
+  float* u = sm + ((36 + S * S + 2 * S + 2 * a.top + 3) & ~3);
+  const size_t t = a.rows ? a.rows[r] : r;
+  const bool update = a.y != nullptr || a.down != nullptr;
+  for (int i = threadIdx.x; i < S * S; i += blockDim.x) mix[i] = update ? a.mix[i] : 0.f;
+  for (int i = threadIdx.x; i < S; i += blockDim.x) {
+    ow[i] = update ? a.out_w[i] : 0.f;
+    iw[i] = a.in_w ? a.in_w[i] : 1.f;
+  }
+  for (int i = threadIdx.x; i < a.top; i += blockDim.x) {
+    cw[i] = a.top_w[t * a.top + i];
+    cr[i] = a.slot_of_pair[t * a.top + i];
+  }
+  __syncthreads();
+  const float* xr = a.x_in + t * width;
+  float sum = 0.f;
+  for (int d = threadIdx.x * V; d < width; d += blockDim.x * V) {
+    FloatVec<V> x[MS], y, acc;
+#pragma unroll
+    for (int s = 0; s < MS; ++s) {
+      if (s >= S) continue;
+      if (s > 0 && a.in_stride == 0) x[s] = x[0];
+      else x[s].load(xr + s * a.in_stride + d);
+    }
+#pragma unroll
+    for (int c = 0; c < V; ++c) acc.v[c] = y.v[c] = 0.f;
+    if (a.down) {
+      for (int j = 0; j < a.top; ++j) {
+        FloatVec<V> e;
+        e.load(a.down + static_cast<size_t>(cr[j]) * width + d);
+#pragma unroll
+        for (int c = 0; c < V; ++c) y.v[c] += cw[j] * e.v[c];
+      }
+    } else if (a.y) {
+      y.load(a.y + t * width + d);
+    }
+#pragma unroll
+    for (int k = 0; k < MS; ++k) {
+      if (k >= S) continue;
+      FloatVec<V> z;
+      if (update) {
+#pragma unroll
+        for (int c = 0; c < V; ++c) z.v[c] = ow[k] * y.v[c];
+#pragma unroll
+        for (int s = 0; s < MS; ++s) {
+          if (s >= S) continue;
+          const float m = mix[s * S + k];
+#pragma unroll
+          for (int c = 0; c < V; ++c) z.v[c] += m * x[s].v[c];
+        }
+      } else {
+        z = x[k];
+      }
+      if (a.x_out) z.store(a.x_out + k * a.out_stride + t * width + d);
+#pragma unroll
+      for (int c = 0; c < V; ++c) acc.v[c] += iw[k] * z.v[c];
+    }
+    if (a.out) {
+      acc.store(u + d);
+#pragma unroll
+      for (int c = 0; c < V; ++c) sum += acc.v[c];
+    }
+  }
+  if (!a.out) return;
+  float mean = 0.f, inv = 1.f;
+  if (a.kind == B200_NORM_LAYER) mean = block_sum(sum, red) / static_cast<float>(width);
+  if (a.kind != B200_NORM_DYNTANH) {
+    float ss = 0.f;
+    for (int d = threadIdx.x * V; d < width; d += blockDim.x * V) {
+      FloatVec<V> f;
+      f.load(u + d);
+#pragma unroll
+      for (int c = 0; c < V; ++c) ss += (f.v[c] - mean) * (f.v[c] - mean);
+    }
+    ss = block_sum(ss, red);
+    inv = 1.f / sqrtf(ss / static_cast<float>(width) + a.eps);
+  }
+  T* o = reinterpret_cast<T*>(a.out) + static_cast<size_t>(r) * width;
+  for (int d = threadIdx.x * V; d < width; d += blockDim.x * V) {      // a thread's own columns: no barrier needed
+    FloatVec<V> f, wv, bv;
+    f.load(u + d);
+    wv.load(a.w + d);
+#pragma unroll
+    for (int c = 0; c < V; ++c) bv.v[c] = 0.f;
+    if (a.bias) bv.load(a.bias + d);
+#pragma unroll
+    for (int c = 0; c < V; ++c)
+      f.v[c] = a.kind == B200_NORM_DYNTANH ? tanhf(a.alpha * f.v[c]) * wv.v[c] + bv.v[c]
+                                           : (f.v[c] - mean) * inv * (a.w_offset + wv.v[c]) + bv.v[c];
+    store_vec<V>(o + d, f);
+  }
+}
+
+// out[i] = sum_j w[j] * hist[j * stride + i] (w == nullptr: ones), V floats per thread and step
 template <int V>
 __global__ void depth_mix_kernel(float* __restrict__ out, const float* __restrict__ hist, size_t stride,
                                  const float* __restrict__ w, int count, size_t n) {
@@ -191,14 +351,14 @@ __global__ void depth_mix_kernel(float* __restrict__ out, const float* __restric
     if constexpr (V == 4) {
       float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int j = 0; j < count; ++j) {
-        const float wj = w[j];
+        const float wj = w ? w[j] : 1.f;
         const float4 v = *reinterpret_cast<const float4*>(hist + j * stride + i * 4);
         acc.x += wj * v.x; acc.y += wj * v.y; acc.z += wj * v.z; acc.w += wj * v.w;
       }
       *reinterpret_cast<float4*>(out + i * 4) = acc;
     } else {
       float acc = 0.f;
-      for (int j = 0; j < count; ++j) acc += w[j] * hist[j * stride + i];
+      for (int j = 0; j < count; ++j) acc += (w ? w[j] : 1.f) * hist[j * stride + i];
       out[i] = acc;
     }
   }
@@ -280,15 +440,19 @@ void launch_silu_mul_f32(void* out, const float* gate_up, int T, int ff, int dt,
   B200_CUDA_LAUNCH_CHECK();
 }
 
-void launch_relu2_f32(void* out, const float* up, int ld, int T, int ff, int gate_col, const float* bias, int dt,
-                      cudaStream_t st_) {
+void launch_ff_act(void* out, const float* up, int ld, int T, int ff, int gate_col, const float* bias, int act, int dt,
+                   cudaStream_t st_) {
   const size_t total = static_cast<size_t>(T) * ff;
   if (total == 0) return;
+  if (act != 1 && act != 2) {
+    set_error(1, "ff_act: unknown activation");
+    return;
+  }
+  auto go = [&](auto* o, auto kern) { kern<<<flat_grid(total), 256, 0, st_>>>(o, up, ld, ff, gate_col, bias, total); };
   if (dt)
-    relu2_f32_kernel<float><<<flat_grid(total), 256, 0, st_>>>((float*)out, up, ld, ff, gate_col, bias, total);
+    go((float*)out, act == 1 ? ff_act_kernel<float, 1> : ff_act_kernel<float, 2>);
   else
-    relu2_f32_kernel<__nv_bfloat16><<<flat_grid(total), 256, 0, st_>>>((__nv_bfloat16*)out, up, ld, ff, gate_col, bias,
-                                                                       total);
+    go((__nv_bfloat16*)out, act == 1 ? ff_act_kernel<__nv_bfloat16, 1> : ff_act_kernel<__nv_bfloat16, 2>);
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -303,6 +467,49 @@ void launch_stream_norm(void* out, const float* x, const float* w, const float* 
   else
     stream_norm_kernel<__nv_bfloat16><<<T, 256, 0, st_>>>((__nv_bfloat16*)out, x, w, bias, alpha, kind, width, eps, w_offset,
                                                           rows, shift_w, shift_state, slots, cu, ctx, num_seqs);
+  B200_CUDA_LAUNCH_CHECK();
+}
+
+template <typename T, int MS>
+static void hyper_step_vec(const HyperArgs& a, int rows, bool vec, size_t smem, cudaStream_t st_) {
+  auto go = [&](auto kern, int threads) {
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    kern<<<rows, threads, smem, st_>>>(a);
+  };
+  if (vec) go(hyper_step_kernel<T, MS, 4>, a.width >= 1024 ? 256 : (a.width >= 512 ? 128 : 64));
+  else go(hyper_step_kernel<T, MS, 1>, 256);
+}
+
+void launch_hyper_step(void* out, float* x_out, size_t out_stride, const float* x_in, size_t in_stride, const float* y,
+                       const float* down, const int32_t* slot_of_pair, const float* top_w, int top, const float* mix,
+                       const float* out_w, const float* in_w, const float* w, const float* bias, float alpha, int kind,
+                       float eps, float w_offset, const uint32_t* rows, int streams, int T, int width, int dt,
+                       cudaStream_t st_) {
+  if (T <= 0) return;
+  if (streams < 1 || streams > B200_MAX_STREAMS) {
+    set_error(1, "hyper_step: 1 to 16 streams");
+    return;
+  }
+  if (!down) top = 0;
+  const HyperArgs a{out, x_out, out_stride, x_in, in_stride, y, down, slot_of_pair, top_w, top, mix, out_w, in_w, w, bias,
+                    alpha, kind, eps, w_offset, rows, streams, width};
+  const size_t smem = (static_cast<size_t>((36 + streams * streams + 2 * streams + 2 * top + 3) & ~3) + width) * 4;
+  if (smem > 220 * 1024) {
+    set_error(1, "hyper_step: rows too wide for shared memory");
+    return;
+  }
+  auto al = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool vec = width % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && al(out) && al(x_out) && al(x_in) && al(y) &&
+                   al(down) && al(w) && al(bias);
+#define B200_HYPER(MS)                                                     \
+  if (dt) hyper_step_vec<float, MS>(a, T, vec, smem, st_);                 \
+  else hyper_step_vec<__nv_bfloat16, MS>(a, T, vec, smem, st_);
+  if (streams == 1) { B200_HYPER(1) }
+  else if (streams == 2) { B200_HYPER(2) }
+  else if (streams <= 4) { B200_HYPER(4) }
+  else if (streams <= 8) { B200_HYPER(8) }
+  else { B200_HYPER(16) }
+#undef B200_HYPER
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -349,16 +556,34 @@ void b200_stream_norm(void* out, const float* x, const float* w, const float* bi
                       float eps, float w_offset, const uint32_t* rows, const float* shift_w, float* shift_state,
                       const int32_t* state_slots, const uint32_t* cu_seqlens_q, const uint32_t* context_lens,
                       int32_t num_seqs, int32_t num_tokens, int32_t width, int32_t dt, int64_t stream) {
-  B200_CHECK_ARG(out && x && w && width > 0 && (dt == 0 || dt == 1) && (kind == B200_NORM_RMS || kind == B200_NORM_DYNTANH) &&
+  B200_CHECK_ARG(out && x && w && width > 0 && (dt == 0 || dt == 1) && kind >= B200_NORM_RMS && kind <= B200_NORM_LAYER &&
                      (!shift_w || (!rows && shift_state && state_slots && cu_seqlens_q && context_lens && num_seqs > 0)),
                  "stream_norm: bad arguments (a token shift needs the step's sequences and a state, and no row list)");
   b200::launch_stream_norm(out, x, w, bias, alpha, kind, eps, w_offset, rows, shift_w, shift_state, state_slots,
                            cu_seqlens_q, context_lens, num_seqs, num_tokens, width, dt,
                            reinterpret_cast<cudaStream_t>(stream));
 }
+void b200_hyper_step(void* out, float* x_out, int64_t out_stride, const float* x_in, int64_t in_stride, const float* y,
+                     const float* down, const int32_t* slot_of_pair, const float* top_w, int32_t top, const float* mix,
+                     const float* out_w, const float* in_w, const float* w, const float* bias, float alpha, int32_t kind,
+                     float eps, float w_offset, const uint32_t* rows, int32_t streams, int32_t num_tokens, int32_t width,
+                     int32_t dt, int64_t stream) {
+  B200_CHECK_ARG((out || x_out) && x_in && width > 0 && (dt == 0 || dt == 1) && in_stride >= 0 && out_stride >= 0 &&
+                     (!out || w) && (!(y || down) || (mix && out_w)) && (!down || (slot_of_pair && top_w && top > 0)) &&
+                     (!rows || !x_out) && kind >= B200_NORM_RMS && kind <= B200_NORM_LAYER,
+                 "hyper_step: bad arguments");
+  b200::launch_hyper_step(out, x_out, static_cast<size_t>(out_stride), x_in, static_cast<size_t>(in_stride), y, down,
+                          slot_of_pair, top_w, top, mix, out_w, in_w, w, bias, alpha, kind, eps, w_offset, rows, streams,
+                          num_tokens, width, dt, reinterpret_cast<cudaStream_t>(stream));
+}
+void b200_ff_act(void* out, const float* up, int32_t ld, const float* bias, int32_t act, int32_t num_tokens, int32_t n,
+                 int32_t dt, int64_t stream) {
+  B200_CHECK_ARG(out && up && n > 0 && ld >= n && (act == 1 || act == 2) && (dt == 0 || dt == 1), "ff_act: bad arguments");
+  b200::launch_ff_act(out, up, ld, num_tokens, n, -1, bias, act, dt, reinterpret_cast<cudaStream_t>(stream));
+}
 void b200_depth_mix(float* out, const float* hist, int64_t stride, const float* w, int32_t count, int64_t n,
                     int64_t stream) {
-  B200_CHECK_ARG(out && hist && w && count > 0 && stride >= 0 && n >= 0, "depth_mix: bad arguments");
+  B200_CHECK_ARG(out && hist && count > 0 && stride >= 0 && n >= 0, "depth_mix: bad arguments");
   b200::launch_depth_mix(out, hist, static_cast<size_t>(stride), w, count, static_cast<size_t>(n),
                          reinterpret_cast<cudaStream_t>(stream));
 }

@@ -84,16 +84,22 @@ void launch_resid_add_rmsnorm(float* x, const float* y, const float* w, int T, i
 void launch_bias_rows(float* y, const float* bias, float scale, int T, int n, cudaStream_t st);
 void launch_cast_rows(void* out, const float* in, int ld_in, int T, int n, int dt, cudaStream_t st);
 void launch_silu_mul_f32(void* out, const float* gate_up, int T, int ff, int dt, cudaStream_t st);
-// out [T, ff] = relu(up[t, d])^2 (* sigmoid(up[t, gate_col]) when gate_col >= 0); up fp32 with row stride ld
-// bias (may be NULL): fp32 [ff], added before the activation
-void launch_relu2_f32(void* out, const float* up, int ld, int T, int ff, int gate_col, const float* bias, int dt,
-                      cudaStream_t st);
+// out [T, ff] = act(up[t, d] + bias[d]) (* sigmoid(up[t, gate_col]) when gate_col >= 0); act 1: relu(.)^2, 2: exact GELU;
+// up fp32 with row stride ld; bias (may be NULL): fp32 [ff]
+void launch_ff_act(void* out, const float* up, int ld, int T, int ff, int gate_col, const float* bias, int act, int dt,
+                   cudaStream_t st);
 // norm of the stream (kind B200_NORM_*), optionally followed by the token shift (see b200_stream_norm)
 void launch_stream_norm(void* out, const float* x, const float* w, const float* bias, float alpha, int kind, float eps,
                         float w_offset, const uint32_t* rows, const float* shift_w, float* shift_state,
                         const int32_t* slots, const uint32_t* cu, const uint32_t* ctx, int num_seqs, int T, int width,
                         int dt, cudaStream_t st);
 void launch_depth_mix(float* out, const float* hist, size_t stride, const float* w, int count, size_t n, cudaStream_t st);
+// the step between two sublayers of hyper-connected streams (see b200_hyper_step)
+void launch_hyper_step(void* out, float* x_out, size_t out_stride, const float* x_in, size_t in_stride, const float* y,
+                       const float* down, const int32_t* slot_of_pair, const float* top_w, int top, const float* mix,
+                       const float* out_w, const float* in_w, const float* w, const float* bias, float alpha, int kind,
+                       float eps, float w_offset, const uint32_t* rows, int streams, int T, int width, int dt,
+                       cudaStream_t st);
 
 void launch_latent_prep(const float* qc, int ldq, void* q_plain, float* q_full, void* cache, const float* latent_norm_w,
                         const double* rot_freq, float rot_mag, const int64_t* positions, const int64_t* slots, int T,
@@ -143,8 +149,9 @@ void launch_decay_attn(float* out, const float* q, const float* k, const float* 
                        const int32_t* slots, const uint32_t* cu, const uint32_t* ctx, int num_seqs, int heads, int dim,
                        int vdim, cudaStream_t st);
 
-void launch_moe_route(const float* logits, const float* bias, int T, int E, int top, int groups, int keep, float scale,
-                      int32_t* top_idx, float* top_w, cudaStream_t st);
+// score 0 softmax, 1 sigmoid; group_top: a group's score sums its 1 or 2 best members; renorm: weights / (their sum + 1e-20)
+void launch_moe_route(const float* logits, const float* bias, int T, int E, int top, int groups, int keep, int score,
+                      int group_top, int renorm, float scale, int32_t* top_idx, float* top_w, cudaStream_t st);
 void launch_moe_sort(const int32_t* top_idx, int pairs, int E, int32_t* expert_off, int32_t* pair_of_slot,
                      int32_t* slot_of_pair, cudaStream_t st);
 // act 0: SiLU(gate) * up over [gate | up] rows; act 1: relu(up)^2 over up rows

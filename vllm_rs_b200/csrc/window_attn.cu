@@ -14,8 +14,10 @@
 //     output element (gate[t, h * vdim + d])
 //   * a distance bias: the score of query position i against key position j is lowered by slope_h * (i - j), after
 //     scale and cap (slopes fp32 per head, NULL: none)
+//   * a learned distance bias: the score gains table[h, min(i - j, n - 1)] (fp32, one value per head and distance, the
+//     last one for everything further away), after scale and cap
 //   * in the prep kernel: q / k norms per head with one weight of size dim shared by the heads (instead of over the
-//     whole projection), values that are the un-normed key rows (no v projection), and a query temperature
+//     whole projection) or without a weight, values mixed with another layer's values of the same token, values that are the un-normed key rows (no v projection), and a query temperature
 //     1 + coef * ln(floor((p + 1) / every) + 1) at position p
 //   * rotary pairs either interleaved (2i, 2i+1) or as the two halves of the rotated part (i, i + rot_dims / 2), with a
 //     factor on cos and sin
@@ -54,7 +56,8 @@ __global__ void window_attn_prep_kernel(const float* __restrict__ proj, int ld, 
                                         T* __restrict__ k_cache, T* __restrict__ v_cache, int heads, int kv_heads,
                                         int dim, int vdim, int rot_dims, float eps, int head_norm, int v_from_k,
                                         int q_temp_every, float q_temp_coef, int rot_half, float rot_mag,
-                                        const double* __restrict__ v_rot_freq, int v_heads) {
+                                        const double* __restrict__ v_rot_freq, int v_heads, float v_mix,
+                                        float* __restrict__ v_first_out, const float* __restrict__ v_first) {
   extern __shared__ float sm[];          // cos[rot_dims/2] | sin[rot_dims/2] | red[36] | hinv[heads + kv_heads] | vcos, vsin[vdim/2]
   const int half = rot_dims / 2, vhalf = vdim / 2;
   float* cs = sm;
@@ -102,7 +105,7 @@ __global__ void window_attn_prep_kernel(const float* __restrict__ proj, int ld, 
         ss += v * v;
       }
       ss = lanes_sum(ss);
-      if (lane == 0) hinv[hh] = (isq ? q_norm_w : k_norm_w) ? 1.f / sqrtf(ss / static_cast<float>(dim) + eps) : 1.f;
+      if (lane == 0) hinv[hh] = (head_norm == 2 || (isq ? q_norm_w : k_norm_w)) ? 1.f / sqrtf(ss / static_cast<float>(dim) + eps) : 1.f;
     }
   } else if (q_norm_w) {
     float ss = 0.f;
@@ -144,14 +147,20 @@ __global__ void window_attn_prep_kernel(const float* __restrict__ proj, int ld, 
   if (slot >= 0 && k_cache) {            // no cache: the row brought queries only
     for (int e = threadIdx.x; e < nk; e += blockDim.x)
       st(k_cache + static_cast<size_t>(slot) * nk + e, entry(kr, bk, k_norm_w, inv_k, heads, e));
+    const float* first = v_first ? v_first + static_cast<size_t>(t) * nv : nullptr;
+    auto value = [&](int e) {            // projection + bias, mixed with the kept values of the same token
+      const float v = vr[e] + (bv ? bv[e] : 0.f);
+      return first ? (1.f - v_mix) * v + v_mix * first[e] : v;
+    };
     for (int e = threadIdx.x; e < nv; e += blockDim.x) {
-      float val = vr[e] + (bv ? bv[e] : 0.f);
+      float val = value(e);
+      if (v_first_out) v_first_out[static_cast<size_t>(t) * nv + e] = val;
       if (v_rot_freq) {                  // the value row turned by its own position, all of vdim
         const int d = e % vdim;
         const bool second = rot_half ? d >= vhalf : (d & 1) != 0;
         const int i = rot_half ? (second ? d - vhalf : d) : d >> 1;
         const int eo = second ? (rot_half ? e - vhalf : e - 1) : (rot_half ? e + vhalf : e + 1);   // the other member
-        const float other = vr[eo] + (bv ? bv[eo] : 0.f);
+        const float other = value(eo);
         val = second ? val * vcs[i] + other * vsn[i] : val * vcs[i] - other * vsn[i];
       }
       st(v_cache + static_cast<size_t>(slot) * nv + e, val);
@@ -193,7 +202,7 @@ __global__ void window_attn_kernel(T* __restrict__ out, const float* __restrict_
                                    int keep_first, float scale, float softcap, int key_tile, int nsplit,
                                    float* __restrict__ part_o, float* __restrict__ part_ml,
                                    const float* __restrict__ slopes, int gate_elems, int chunk, int v_heads,
-                                   int out_f32) {
+                                   int out_f32, const float* __restrict__ dist_bias, int dist_n) {
   extern __shared__ float sm[];
   const int Dp = dim | 1;                               // odd row pitch: a lane per key reads conflict-free
   const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -252,7 +261,9 @@ __global__ void window_attn_kernel(T* __restrict__ out, const float* __restrict_
           const float* kr = ks + k * Dp;
           const float* qw = qs + warp * dim;
           for (int d = 0; d < dim; ++d) acc += qw[d] * kr[d];
-          s = cap_score(acc * scale, softcap) - slope * static_cast<float>(pos - vis.key(i0 + k));
+          const int dist = pos - vis.key(i0 + k);
+          s = cap_score(acc * scale, softcap) - slope * static_cast<float>(dist);
+          if (dist_bias) s += dist_bias[static_cast<size_t>(h) * dist_n + min(dist, dist_n - 1)];
         }
         const float mt = lanes_max(s);
         const float mn = fmaxf(m, mt);
@@ -326,6 +337,13 @@ void launch_window_attn_prep(const float* proj, int ld, const float* bias, const
   const float rot_mag = (opt && opt->rot_mag != 0.f) ? opt->rot_mag : 1.f;
   const double* v_rot = opt ? opt->v_rot_freq : nullptr;
   const int v_heads = (opt && opt->v_heads > 0) ? opt->v_heads : kv_heads;
+  const float v_mix = opt ? opt->v_mix : 0.f;
+  float* v_first_out = opt ? opt->v_first_out : nullptr;
+  const float* v_first = opt ? opt->v_first : nullptr;
+  if (v_first && v_first_out) {
+    set_error(1, "window_attn_prep: a layer either keeps its values or mixes kept ones in");
+    return;
+  }
   if (opt && opt->no_cache) k_cache = v_cache = nullptr;
   if (v_from_k && (vdim != dim || v_heads != kv_heads)) {
     set_error(1, "window_attn_prep: values taken from the key rows need vdim == dim and as many value heads as key heads");
@@ -340,13 +358,14 @@ void launch_window_attn_prep(const float* proj, int ld, const float* bias, const
     window_attn_prep_kernel<float><<<T, 256, smem, st_>>>(proj, ld, bias, q_norm_w, k_norm_w, rot_freq, positions, slots,
                                                           q_out, (float*)k_cache, (float*)v_cache, heads, kv_heads, dim,
                                                           vdim, rot_dims, eps, head_norm, v_from_k, q_every, q_coef,
-                                                          rot_half, rot_mag, v_rot, v_heads);
+                                                          rot_half, rot_mag, v_rot, v_heads, v_mix, v_first_out, v_first);
   else
     window_attn_prep_kernel<__nv_bfloat16><<<T, 256, smem, st_>>>(proj, ld, bias, q_norm_w, k_norm_w, rot_freq, positions,
                                                                   slots, q_out, (__nv_bfloat16*)k_cache,
                                                                   (__nv_bfloat16*)v_cache, heads, kv_heads, dim, vdim,
                                                                   rot_dims, eps, head_norm, v_from_k, q_every, q_coef,
-                                                                  rot_half, rot_mag, v_rot, v_heads);
+                                                                  rot_half, rot_mag, v_rot, v_heads, v_mix, v_first_out,
+                                                                  v_first);
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -384,7 +403,8 @@ window_attn_mma_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict_
                        const uint32_t* __restrict__ block_tables, int max_blocks, int num_seqs, int heads, int kv_heads,
                        int dim, int vdim, int window, int keep_first, float scale, float softcap, int nsplit,
                        float* __restrict__ part_o, float* __restrict__ part_ml, const float* __restrict__ slopes,
-                       int gate_elems, int chunk, int v_heads, int out_f32) {
+                       int gate_elems, int chunk, int v_heads, int out_f32, const float* __restrict__ dist_bias,
+                       int dist_n) {
   extern __shared__ __align__(16) unsigned char smraw[];
   const int P = dim + 8, PV = vdim + 8;                   // row pitches in bf16 elements (16-byte multiples)
   // maps whose K tiles a block stages: all of them in the heads-as-rows form, the one of the block's head otherwise
@@ -434,7 +454,8 @@ window_attn_mma_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict_
     const float v = r < nrows ? q[qrow * dim + d] : 0.f;
     Qs[r * P + d] = __float2bfloat16_rn(v);
   }
-  float m[2], l[2], slope[2];
+  float m[2], l[2], slope[2], far_bias[2] = {0.f, 0.f};
+  const float* near_bias[2] = {nullptr, nullptr};          // this lane's rows' tables of the distance bias
 #pragma unroll
   for (int rr = 0; rr < 2; ++rr) {
     const int hh = HROWS ? head_of(min(g + rr * 8, nrows - 1)) : h;
@@ -442,6 +463,10 @@ window_attn_mma_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict_
     m[rr] = with_sink ? sink[hh] : -1e30f;
     l[rr] = with_sink ? 1.f : 0.f;
     slope[rr] = slopes ? slopes[hh] : 0.f;
+    if (dist_bias) {
+      near_bias[rr] = dist_bias + static_cast<size_t>(hh) * dist_n;
+      far_bias[rr] = near_bias[rr][dist_n - 1];
+    }
   }
   float o[NT][4];
 #pragma unroll
@@ -511,6 +536,8 @@ window_attn_mma_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict_
     // the same online softmax in every warp; this lane's P entries are exactly its A fragments
     float p[2][16];
     float mx[2] = {-1e30f, -1e30f};
+    // does any key of the tile lie nearer than the table's last entry (which holds for everything further away)?
+    const bool near = dist_bias && pos0 - (HROWS ? tile_key(WKT - 1) : j0 + WKT - 1) < dist_n - 1;
 #pragma unroll
     for (int rr = 0; rr < 2; ++rr) {
       const int r = g + rr * 8;
@@ -522,7 +549,9 @@ window_attn_mma_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict_
           const int kcol = ks * 16 + 2 * tq + (c & 1) + (c >> 1) * 8, j = j0 + kcol;
           const bool ok = HROWS ? (r < nrows && j < t_end) : (r < nrows && j <= rowp[rr] && (j >= lo || j < keep_first));
           const int jpos = HROWS ? vis.key(min(j, t_end - 1)) : j;         // the key's position
-          const float v = ok ? Ss[r * (WKT + 1) + kcol] - slope[rr] * static_cast<float>(rowp[rr] - jpos) : -1e30f;
+          const int dist = rowp[rr] - jpos;
+          float v = ok ? Ss[r * (WKT + 1) + kcol] - slope[rr] * static_cast<float>(dist) : -1e30f;
+          if (ok) v += near ? near_bias[rr][min(dist, dist_n - 1)] : far_bias[rr];
           p[rr][ks * 4 + c] = v;
           mx[rr] = fmaxf(mx[rr], v);
         }
@@ -628,12 +657,14 @@ window_attn_rows_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict
                         const uint32_t* __restrict__ cu, const uint32_t* __restrict__ ctx,
                         const uint32_t* __restrict__ block_tables, int max_blocks, int num_seqs, int heads, int kv_heads,
                         int dim, int vdim, int window, int keep_first, float scale, float softcap,
-                        const float* __restrict__ slopes, int gate_elems, int chunk, int v_heads, int out_f32) {
+                        const float* __restrict__ slopes, int gate_elems, int chunk, int v_heads, int out_f32,
+                        const float* __restrict__ dist_bias, int dist_n, int stage_bias) {
   extern __shared__ __align__(16) unsigned char smraw[];
   const int P = dim + 8, PV = vdim + 8;
   __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smraw);              // [WKT][P]
   __nv_bfloat16* Vs = Ks + static_cast<size_t>(WKT) * P;                    // [WKT][PV]
   __nv_bfloat16* Qs = Vs + static_cast<size_t>(WKT) * PV;                   // [RQ][P]
+  float* bias_s = reinterpret_cast<float*>(Qs + static_cast<size_t>(RQ) * P);   // [dist_n] when stage_bias
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
   int b = -1, row0 = 0, nrows = 0;
   {
@@ -653,6 +684,12 @@ window_attn_rows_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict
   }
   const int h = blockIdx.y, kvh = h / (heads / kv_heads), vh = kvh % v_heads;
   const float slope = slopes ? slopes[h] : 0.f;
+  const float* near_bias = dist_bias ? dist_bias + static_cast<size_t>(h) * dist_n : nullptr;
+  const float far_bias = dist_bias ? near_bias[dist_n - 1] : 0.f;
+  if (stage_bias) {                        // (read behind the barriers of the first tile)
+    for (int i = threadIdx.x; i < dist_n; i += blockDim.x) bias_s[i] = near_bias[i];
+    near_bias = bias_s;
+  }
   const int pos0 = static_cast<int>(ctx[b]) - static_cast<int>(cu[b + 1] - cu[b]) + (row0 - static_cast<int>(cu[b]));
   const int pos_last = pos0 + nrows - 1;
   const int key_lo = first_visible(pos0, window, chunk);
@@ -725,8 +762,25 @@ window_attn_rows_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict
         wmma_bf16_16816(sc[2 * np + 1], a, r2, r3);
       }
     }
-    // scale, cap, mask; row maxima over the lane's entries and the quad
+    // scale, cap, distance bias, mask; row maxima over the lane's entries and the quad.  The table of the distance bias is
+    // read only where a key of the tile lies nearer to the warp's first row than the table's last entry.
     float mx[2] = {-1e30f, -1e30f};
+    if (dist_bias && w_first - (j0 + WKT - 1) < dist_n - 1) {
+#pragma unroll
+      for (int rr = 0; rr < 2; ++rr)
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const int dist = rowp[rr] - (j0 + n * 8 + 2 * tq + c);
+            sc[n][rr * 2 + c] = cap_score(sc[n][rr * 2 + c] * scale, softcap) + near_bias[max(0, min(dist, dist_n - 1))];
+          }
+    } else {
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) sc[n][c] = cap_score(sc[n][c] * scale, softcap) + far_bias;
+    }
 #pragma unroll
     for (int rr = 0; rr < 2; ++rr) {
       const int lo = first_visible(rowp[rr], window, chunk);
@@ -736,8 +790,7 @@ window_attn_rows_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict
         for (int c = 0; c < 2; ++c) {
           const int j = j0 + n * 8 + 2 * tq + c;
           const bool ok = rowi[rr] < nrows && j <= rowp[rr] && (j >= lo || j < keep_first);
-          const float v = ok ? cap_score(sc[n][rr * 2 + c] * scale, softcap) - slope * static_cast<float>(rowp[rr] - j)
-                             : -1e30f;
+          const float v = ok ? sc[n][rr * 2 + c] - slope * static_cast<float>(rowp[rr] - j) : -1e30f;
           sc[n][rr * 2 + c] = v;
           mx[rr] = fmaxf(mx[rr], v);
         }
@@ -875,6 +928,12 @@ void launch_window_attn(void* out, const float* q, const void* k_cache, const vo
   const float* slopes = opt ? opt->dist_slopes : nullptr;
   const int gate_elems = opt ? opt->gate_elems : 0;
   const int chunk = opt ? opt->chunk : 0, out_f32 = opt ? opt->out_f32 : 0;
+  const float* dist_bias = opt ? opt->dist_bias : nullptr;
+  const int dist_n = opt ? opt->dist_n : 0;
+  if (dist_bias && dist_n < 1) {
+    set_error(1, "window_attn: an empty table of the distance bias");
+    return;
+  }
   const int v_heads = (opt && opt->v_heads > 0) ? opt->v_heads : kv_heads;
   if (kv_heads % v_heads != 0) {
     set_error(1, "window_attn: kv_heads is a multiple of v_heads");
@@ -883,7 +942,9 @@ void launch_window_attn(void* out, const float* q, const void* k_cache, const vo
   // bf16, steps of many rows, value sizes up to 128: the tensor-core form with 64 token rows per block
   if (!dt && window_mma_enabled() && T > 2 * sm_count() / 4 && window_rows_enabled() && dim % 16 == 0 && vdim % 16 == 0 &&
       vdim <= 128) {
-    const size_t smem = (static_cast<size_t>(WKT + RQ) * (dim + 8) + static_cast<size_t>(WKT) * (vdim + 8)) * 2;
+    const int stage_bias = dist_bias && dist_n <= 2048;
+    const size_t smem = (static_cast<size_t>(WKT + RQ) * (dim + 8) + static_cast<size_t>(WKT) * (vdim + 8)) * 2 +
+                        (stage_bias ? static_cast<size_t>(dist_n) * 4 : 0);
     const dim3 grid((T + RQ - 1) / RQ + num_seqs, heads, 1);
 #define B200_WROWS(NTV)                                                                                           \
   {                                                                                                                \
@@ -892,7 +953,8 @@ void launch_window_attn(void* out, const float* q, const void* k_cache, const vo
     kern<<<grid, 128, smem, st_>>>((__nv_bfloat16*)out, q, (const __nv_bfloat16*)k_cache,                          \
                                    (const __nv_bfloat16*)v_cache, sink, gate, ld_gate, cu, ctx, block_tables,      \
                                    max_blocks, num_seqs, heads, kv_heads, dim, vdim, window, keep_first, scale,    \
-                                   softcap, slopes, gate_elems, chunk, v_heads, out_f32);                          \
+                                   softcap, slopes, gate_elems, chunk, v_heads, out_f32, dist_bias, dist_n,        \
+                                   stage_bias);                                                                    \
   }
     bool done = smem <= 200 * 1024;
     if (done) switch (vdim / 8) {
@@ -928,7 +990,8 @@ void launch_window_attn(void* out, const float* q, const void* k_cache, const vo
     kern<<<grid, 128, smem, st_>>>((__nv_bfloat16*)out, q, (const __nv_bfloat16*)k_cache,                          \
                                    (const __nv_bfloat16*)v_cache, sink, gate, ld_gate, cu, ctx, block_tables,      \
                                    max_blocks, num_seqs, heads, kv_heads, dim, vdim, window, keep_first, scale,    \
-                                   softcap, nsplit, part_o, part_ml, slopes, gate_elems, chunk, v_heads, out_f32); \
+                                   softcap, nsplit, part_o, part_ml, slopes, gate_elems, chunk, v_heads, out_f32,  \
+                                   dist_bias, dist_n);                                                             \
   }
 #define B200_WMMA(NT)                 \
   if (hrows) B200_WMMA2(NT, true)     \
@@ -980,7 +1043,7 @@ void launch_window_attn(void* out, const float* q, const void* k_cache, const vo
     kern<<<grid, nw * 32, smem, st_>>>((float*)out, q, (const float*)k_cache, (const float*)v_cache, sink, gate, ld_gate,
                                        cu, ctx, block_tables, max_blocks, num_seqs, heads, kv_heads, dim, vdim, window,
                                        keep_first, scale, softcap, key_tile, nsplit, part_o, part_ml, slopes, gate_elems,
-                                       chunk, v_heads, out_f32);
+                                       chunk, v_heads, out_f32, dist_bias, dist_n);
   } else {
     auto kern = window_attn_kernel<__nv_bfloat16>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
@@ -988,7 +1051,7 @@ void launch_window_attn(void* out, const float* q, const void* k_cache, const vo
                                        (const __nv_bfloat16*)v_cache, sink, gate, ld_gate, cu, ctx, block_tables,
                                        max_blocks, num_seqs, heads, kv_heads, dim, vdim, window, keep_first, scale,
                                        softcap, key_tile, nsplit, part_o, part_ml, slopes, gate_elems, chunk, v_heads,
-                                       out_f32);
+                                       out_f32, dist_bias, dist_n);
   }
   B200_CUDA_LAUNCH_CHECK();
   if (nsplit > 1) {

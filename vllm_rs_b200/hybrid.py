@@ -2,8 +2,9 @@
 csrc/host/hybrid_runner.cpp): the sibling of engine.ModelRunner for models whose layers choose between latent
 attention, windowed softmax attention, the gated delta rule, the SSD scan and decayed linear attention (one mixer, or
 two side by side), with a routed mixture of experts or a dense feed-forward, in a parallel, a sandwich
-(norm before and after each sublayer), a post-norm (sublayer results normed on their way into the stream) or a
-pre-norm layout (RMS or dynamic-tanh norms, optional token shift and depth-weighted average of the layers' results).
+(norm before and after each sublayer), a post-norm (sublayer results normed on their way into the stream), a pre-norm
+(RMS, layer or dynamic-tanh norms, optional token shift and depth-weighted average of the layers' results) or a
+hyper-connected layout (pre-norm sublayers that read and rewrite several residual streams).
 
 This module holds no model arithmetic.  It allocates what the C side borrows -- the paged latent caches, the
 paged K / V caches, the slot-indexed recurrent state pools, the workspace, pinned staging -- describes the layers to it, and moves a step's
@@ -21,8 +22,9 @@ from . import _lib
 from ._lib import HybridConfig, HybridLayer
 
 MIXER_LATENT_ATTN, MIXER_DELTA_RULE, MIXER_SSD, MIXER_WINDOW_ATTN, MIXER_DECAY_ATTN = 0, 1, 2, 3, 4
-LAYOUT_PARALLEL, LAYOUT_SANDWICH, LAYOUT_POSTNORM, LAYOUT_PRENORM = 0, 1, 2, 3
-NORM_RMS, NORM_DYNTANH = 0, 1
+LAYOUT_PARALLEL, LAYOUT_SANDWICH, LAYOUT_POSTNORM, LAYOUT_PRENORM, LAYOUT_HYPER = 0, 1, 2, 3, 4
+NORM_RMS, NORM_DYNTANH, NORM_LAYER = 0, 1, 2
+MAX_STREAMS = 16
 PAGE = 64
 
 
@@ -41,7 +43,7 @@ class HybridRunner:
     def __init__(self, *, width, vocab, layers: list[LayerSpec], embed, final_norm, lm_head, norm_eps,
                  norm_weight_offset=0.0, embed_scale=1.0, embed_pos_base=0.0, dtype=torch.bfloat16, num_blocks, max_blocks_per_seq, max_seqs, max_tokens,
                  num_state_slots, device="cuda", layer_trace=False, final_norm_kind=NORM_RMS, final_norm_bias=None,
-                 final_norm_alpha=1.0):
+                 final_norm_alpha=1.0, streams=0):
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("hybrid decoders run with bfloat16 or float32 operands")
         self._l = _lib.lib()
@@ -51,7 +53,7 @@ class HybridRunner:
                                 block_size=PAGE, num_blocks=num_blocks, max_blocks_per_seq=max_blocks_per_seq,
                                 max_seqs=max_seqs, max_tokens=max_tokens, num_state_slots=num_state_slots,
                                 norm_eps=norm_eps, norm_weight_offset=norm_weight_offset, embed_scale=embed_scale,
-                                embed_pos_base=embed_pos_base, final_norm_kind=final_norm_kind)
+                                embed_pos_base=embed_pos_base, final_norm_kind=final_norm_kind, streams=streams)
         self._h = self._l.b200_hybrid_new(C.byref(self.cfg))
         _lib.check()
         self._keep = [embed, final_norm, lm_head, final_norm_bias]
