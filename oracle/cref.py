@@ -1,7 +1,7 @@
 """ctypes wrapper + build recipe for oracle/c/decode_ref.c (CPU baseline / C restatement).
 
 TEST INFRASTRUCTURE (see oracle/__init__.py).  Output goes to oracle/_build/ (git-ignored,
-travels to the GPU box with gpurun like the product .so).
+built in-tree like the product .so).
 """
 from __future__ import annotations
 

@@ -1,4 +1,4 @@
-"""Multi-GPU (needs >= 2 B200s: `gpurun --gpus 2`): the communicator (NCCL baseline and the
+"""Multi-GPU (needs >= 2 B200s): the communicator (NCCL baseline and the
 one-shot NVLink all-reduce, eager and inside a CUDA graph) and a TP=2 sharded decode step vs the
 unsharded CPU oracle.  One process per GPU, like the reference's runner processes."""
 import os

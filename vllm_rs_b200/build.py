@@ -4,7 +4,7 @@
     python -m vllm_rs_b200.build --force
     python -m vllm_rs_b200.build --target hybrid
 
-Output: vllm_rs_b200/libb200_vllm.so (git-ignored; travels to the GPU box with gpurun).  The `hybrid` target builds
+Output: vllm_rs_b200/libb200_vllm.so (git-ignored).  The `hybrid` target builds
 vllm_rs_b200/libb200_hybrid.so from the sources the fp32-residual hybrid decoders need and nothing else (no tcgen05
 GEMM / attention kernels): what a fresh checkout compiles when it is first asked to serve such a model.
 """
