@@ -79,10 +79,12 @@ def random_tensors(cfg, seed=0):
             F = mlp["ff"]
             out.update({q + "gate": lin(F, D), q + "up": lin(F, D), q + "down": lin(D, F)})
         else:
-            r, F, Fs = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+            r, F = mlp["router"], mlp["expert"]["ff"]
             out.update({q + "router": lin(r["experts"] + r["identity"], D),
-                        q + "correction": vec(r["experts"] + r["identity"], 0.0, 0.02),
-                        q + "shared.up": lin(Fs, D), q + "shared.down": lin(D, Fs), q + "shared.sg": lin(1, D)})
+                        q + "correction": vec(r["experts"] + r["identity"], 0.0, 0.02)})
+            if mlp.get("shared"):
+                Fs = mlp["shared"]["ff"]
+                out.update({q + "shared.up": lin(Fs, D), q + "shared.down": lin(D, Fs), q + "shared.sg": lin(1, D)})
             for e in range(r["experts"]):
                 out.update({f"{q}e{e}.up": lin(F, D), f"{q}e{e}.down": lin(D, F)})
     return out

@@ -7,6 +7,8 @@
 // dtype is bf16 or fp32.  Beside the fp16 / bf16 row kernels of glue.cu (rmsnorm_kernel, silu_mul_kernel), which
 // keep a 16-bit residual.
 #include "../../include/b200_vllm.h"
+#include <algorithm>
+
 #include "seqmix.cuh"
 
 namespace b200 {
@@ -122,21 +124,53 @@ __global__ void silu_mul_f32_kernel(T* __restrict__ out, const float* __restrict
   }
 }
 
-// out[t, d] = act(up[t, d] + bias[d]) (* sigmoid(up[t, gate_col]) when gate_col >= 0); ACT 1: relu(.)^2, 2: the exact GELU
-template <typename T, int ACT>
+// V consecutive fp32 values of a thread (16-byte accesses for V = 4), stored as fp32 or rounded to bf16
+template <int V> struct FloatVec;
+template <> struct FloatVec<1> {
+  float v[1];
+  __device__ __forceinline__ void load(const float* p) { v[0] = *p; }
+  __device__ __forceinline__ void store(float* p) const { *p = v[0]; }
+};
+template <> struct FloatVec<4> {
+  float v[4];
+  __device__ __forceinline__ void load(const float* p) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+  }
+  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+};
+template <int V> __device__ __forceinline__ void store_vec(float* p, const FloatVec<V>& f) { f.store(p); }
+template <int V> __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const FloatVec<V>& f) {
+  if constexpr (V == 4) {
+    __nv_bfloat162 q[2] = {__floats2bfloat162_rn(f.v[0], f.v[1]), __floats2bfloat162_rn(f.v[2], f.v[3])};
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(q);
+  } else {
+    *p = __float2bfloat16_rn(f.v[0]);
+  }
+}
+
+// out[t, d] = act(up[t, d] + bias[d]) (* sigmoid(up[t, gate_col]) when gate_col >= 0); ACT 1: relu(.)^2, 2: the exact GELU.
+// grid.x covers the columns (V per thread), grid.y the rows
+template <typename T, int ACT, int V>
 __global__ void ff_act_kernel(T* __restrict__ out, const float* __restrict__ up, int ld, int ff, int gate_col,
-                              const float* __restrict__ bias, size_t total) {
-  for (size_t i = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; i < total;
-       i += static_cast<size_t>(gridDim.x) * blockDim.x) {
-    const size_t t = i / ff, d = i % ff;
-    const float z = up[t * ld + d] + (bias ? bias[d] : 0.f);
-    const float g = gate_col >= 0 ? sigmoid_f(up[t * ld + gate_col]) : 1.f;
-    if (ACT == 1) {
-      const float u = fmaxf(z, 0.f);
-      st(out + i, u * u * g);
-    } else {
-      st(out + i, 0.5f * z * (1.f + erff(z * 0.70710678118654752f)) * g);
+                              const float* __restrict__ bias, int rows) {
+  const int d = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (d >= ff) return;
+  FloatVec<V> b;
+#pragma unroll
+  for (int c = 0; c < V; ++c) b.v[c] = 0.f;
+  if (bias) b.load(bias + d);
+  for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+    const float* row = up + static_cast<size_t>(t) * ld;
+    const float g = gate_col >= 0 ? sigmoid_f(row[gate_col]) : 1.f;
+    FloatVec<V> z;
+    z.load(row + d);
+#pragma unroll
+    for (int c = 0; c < V; ++c) {
+      const float v = z.v[c] + b.v[c], r = fmaxf(v, 0.f);
+      z.v[c] = (ACT == 1 ? r * r : 0.5f * v * (1.f + erff(v * 0.70710678118654752f))) * g;
     }
+    store_vec<V>(out + static_cast<size_t>(t) * ff + d, z);
   }
 }
 
@@ -216,29 +250,6 @@ struct HyperArgs {
   const uint32_t* rows;
   int streams, width;
 };
-template <int V> struct FloatVec;
-template <> struct FloatVec<1> {
-  float v[1];
-  __device__ __forceinline__ void load(const float* p) { v[0] = *p; }
-  __device__ __forceinline__ void store(float* p) const { *p = v[0]; }
-};
-template <> struct FloatVec<4> {
-  float v[4];
-  __device__ __forceinline__ void load(const float* p) {
-    const float4 q = *reinterpret_cast<const float4*>(p);
-    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
-  }
-  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
-};
-template <int V> __device__ __forceinline__ void store_vec(float* p, const FloatVec<V>& f) { f.store(p); }
-template <int V> __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const FloatVec<V>& f) {
-  if constexpr (V == 4) {
-    __nv_bfloat162 q[2] = {__floats2bfloat162_rn(f.v[0], f.v[1]), __floats2bfloat162_rn(f.v[2], f.v[3])};
-    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(q);
-  } else {
-    *p = __float2bfloat16_rn(f.v[0]);
-  }
-}
 template <typename T, int MS, int V>
 __global__ void hyper_step_kernel(const HyperArgs a) {
   // red[36] | mix[S * S] | out_w[S] | in_w[S] | choice weights[top] | choice rows[top] | u[width] (16-byte aligned)
@@ -442,17 +453,21 @@ void launch_silu_mul_f32(void* out, const float* gate_up, int T, int ff, int dt,
 
 void launch_ff_act(void* out, const float* up, int ld, int T, int ff, int gate_col, const float* bias, int act, int dt,
                    cudaStream_t st_) {
-  const size_t total = static_cast<size_t>(T) * ff;
-  if (total == 0) return;
+  if (T <= 0 || ff <= 0) return;
   if (act != 1 && act != 2) {
     set_error(1, "ff_act: unknown activation");
     return;
   }
-  auto go = [&](auto* o, auto kern) { kern<<<flat_grid(total), 256, 0, st_>>>(o, up, ld, ff, gate_col, bias, total); };
-  if (dt)
-    go((float*)out, act == 1 ? ff_act_kernel<float, 1> : ff_act_kernel<float, 2>);
-  else
-    go((__nv_bfloat16*)out, act == 1 ? ff_act_kernel<__nv_bfloat16, 1> : ff_act_kernel<__nv_bfloat16, 2>);
+  const bool vec = ff % 4 == 0 && ld % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(bias)) % 16 == 0;
+  const int per_block = 256 * (vec ? 4 : 1);
+  const dim3 grid((ff + per_block - 1) / per_block, std::min(T, 32768));
+  auto go = [&](auto* o, auto kern) { kern<<<grid, 256, 0, st_>>>(o, up, ld, ff, gate_col, bias, T); };
+#define B200_FF_ACT(TYPE)                                                                     \
+  if (vec) go((TYPE*)out, act == 1 ? ff_act_kernel<TYPE, 1, 4> : ff_act_kernel<TYPE, 2, 4>);   \
+  else go((TYPE*)out, act == 1 ? ff_act_kernel<TYPE, 1, 1> : ff_act_kernel<TYPE, 2, 1>);
+  if (dt) { B200_FF_ACT(float) } else { B200_FF_ACT(__nv_bfloat16) }
+#undef B200_FF_ACT
   B200_CUDA_LAUNCH_CHECK();
 }
 

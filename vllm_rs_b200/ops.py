@@ -467,6 +467,39 @@ def moe_route_ex(logits, bias, top, scale=1.0, groups=0, keep=0):
     return idx, w
 
 
+def moe_route_full(logits, bias, top, scale=1.0, groups=0, keep=0, score="softmax", group_top=1, renorm=False):
+    """The router with every option: score "softmax" or "sigmoid", groups ranked by the sum of their `group_top` (1 or 2)
+    best choice scores, chosen weights divided by their sum (renorm); see b200_moe_route_full."""
+    _cuda(logits, bias)
+    T, E = logits.shape
+    idx = torch.empty(T, top, dtype=torch.int32, device=logits.device)
+    w = torch.empty(T, top, dtype=torch.float32, device=logits.device)
+    _lib.lib().b200_moe_route_full(_p(logits), _p(bias), T, E, int(top), int(groups), int(keep),
+                                   {"softmax": 0, "sigmoid": 1}[score], int(group_top), int(bool(renorm)), float(scale),
+                                   _p(idx), _p(w), _stream())
+    _lib.check()
+    return idx, w
+
+
+def moe_experts_rows(h, top_idx, w_up, w_down, *, act="silu_gate"):
+    """The chosen experts' output rows, unsummed: (rows fp32 [T * top, D] in bucket order, i32 [T * top]: the row of pair
+    token * top + choice)."""
+    _cuda(h, top_idx, w_up, w_down)
+    T, D = h.shape
+    E, rows, _ = w_up.shape
+    F = rows // 2 if act == "silu_gate" else rows
+    top = top_idx.shape[1]
+    nbytes = _lib.lib().b200_moe_workspace_bytes(T, E, top, D, F)
+    ws = torch.empty(nbytes, dtype=torch.uint8, device=h.device)
+    down, slot = C.c_void_p(), C.c_void_p()
+    _lib.lib().b200_moe_experts_rows(_p(h), _p(top_idx), _p(w_up), _p(w_down), T, E, top, D, F,
+                                     {"silu_gate": 0, "relu2": 1}[act], _dt(h.dtype), _p(ws), C.byref(down), C.byref(slot),
+                                     _stream())
+    _lib.check()
+    at, base = lambda p, n, dt: ws[p.value - base:p.value - base + n * 4].view(dt), ws.data_ptr()
+    return at(down, T * top * D, torch.float32).reshape(T * top, D), at(slot, T * top, torch.int32)
+
+
 def moe_experts_ex(out, h, top_idx, top_w, w_up, w_down, *, act="silu_gate", identity=0, accumulate=True, ident=None):
     """out fp32 [T, D] (+)= the chosen experts of h [T, D]; act "silu_gate": w_up [E, 2 F, D]; "relu2": w_up [E, F, D];
     indices >= E are identity experts and return the rows of `ident` (fp32 or h's dtype; default h)."""
@@ -494,34 +527,40 @@ def resid_add_rmsnorm(x, y, w, eps, w_offset=0.0):
 
 
 def _attn_options(head_norm=False, v_from_k=False, q_temp=None, dist_slopes=None, gate_elems=False, rot_half=False,
-                  rot_mag=1.0, v_rot_freq=None, v_heads=0, chunk=0, out_f32=False, no_cache=False):
+                  rot_mag=1.0, v_rot_freq=None, v_heads=0, chunk=0, out_f32=False, no_cache=False, dist_bias=None, v_mix=0.0,
+                  v_first_out=None, v_first=None):
     """b200_attn_options; q_temp = (coef, every) or None.  Keep the returned object alive during the call."""
-    o = _lib.AttnOptions(head_norm=int(bool(head_norm)), v_from_k=int(bool(v_from_k)),
+    ptr = lambda t: t.data_ptr() if t is not None else None      # noqa: E731
+    o = _lib.AttnOptions(head_norm=int(head_norm), v_from_k=int(bool(v_from_k)),
                          q_temp_every=int(q_temp[1]) if q_temp else 0, gate_elems=int(bool(gate_elems)),
                          q_temp_coef=float(q_temp[0]) if q_temp else 0.0,
                          dist_slopes=dist_slopes.data_ptr() if dist_slopes is not None else None,
                          rot_half=int(bool(rot_half)), rot_mag=float(rot_mag),
                          v_rot_freq=v_rot_freq.data_ptr() if v_rot_freq is not None else None, v_heads=int(v_heads),
-                         chunk=int(chunk), out_f32=int(bool(out_f32)), no_cache=int(bool(no_cache)))
+                         chunk=int(chunk), out_f32=int(bool(out_f32)), no_cache=int(bool(no_cache)),
+                         dist_bias=ptr(dist_bias), dist_n=dist_bias.shape[1] if dist_bias is not None else 0,
+                         v_mix=float(v_mix), v_first_out=ptr(v_first_out), v_first=ptr(v_first))
     return o
 
 
 def window_attn_prep(proj, bias, q_norm_w, k_norm_w, rot_freq, positions, slot_mapping, k_cache, v_cache, *, heads,
                      rot_dims, eps, head_norm=False, v_from_k=False, q_temp=None, rot_half=False, rot_mag=1.0,
-                     v_rot_freq=None):
+                     v_rot_freq=None, v_mix=0.0, v_first_out=None, v_first=None):
     """proj fp32 [T, >= heads dim + kv_heads (dim + vdim)] -> q fp32 [T, heads, dim]; writes the K / V cache rows
     (k_cache [blocks, 64, kv_heads, dim], v_cache [blocks, 64, kv_heads, vdim]).  head_norm: q_norm_w / k_norm_w are
     [dim] and every head is normed on its own; v_from_k: no v block, the raw key rows are the values; q_temp =
     (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  rot_half: rotary
     pairs are (i, i + rot_dims / 2); rot_mag multiplies cos and sin; v_rot_freq f64 [vdim / 2]: the value rows are
     rotated by their position over all of vdim.  The value cache may have fewer heads than the key cache (several score
-    maps over one set of values)."""
-    _cuda(proj, bias, q_norm_w, k_norm_w, rot_freq, positions, slot_mapping, k_cache, v_cache, v_rot_freq)
+    maps over one set of values).  head_norm=2: every head is normed on its own, without a weight.  v_first_out fp32
+    [T, v_heads vdim] receives the value rows; with v_first they become (1 - v_mix) v + v_mix v_first."""
+    _cuda(proj, bias, q_norm_w, k_norm_w, rot_freq, positions, slot_mapping, k_cache, v_cache, v_rot_freq, v_first_out,
+          v_first)
     T = proj.shape[0]
     G, dk, dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
     q = torch.empty(T, heads, dk, dtype=torch.float32, device=proj.device)
     opt = _attn_options(head_norm, v_from_k, q_temp, rot_half=rot_half, rot_mag=rot_mag, v_rot_freq=v_rot_freq,
-                        v_heads=v_cache.shape[2])
+                        v_heads=v_cache.shape[2], v_mix=v_mix, v_first_out=v_first_out, v_first=v_first)
     _lib.lib().b200_window_attn_prep_ex(_p(proj), proj.shape[1], _p(bias), _p(q_norm_w), _p(k_norm_w), _p(rot_freq),
                                         _p(positions), _p(slot_mapping), _p(q), _p(k_cache), _p(v_cache), T, heads, G, dk,
                                         dv, int(rot_dims), float(eps), _dt(k_cache.dtype), C.byref(opt), _stream())
@@ -530,12 +569,12 @@ def window_attn_prep(proj, bias, q_norm_w, k_norm_w, rot_freq, positions, slot_m
 
 
 def window_attn(q, k_cache, v_cache, sink, gate, cu_seqlens_q, context_lens, block_tables, *, window, keep_first, scale,
-                softcap=0.0, split=True, dist_slopes=None, chunk=0, out_f32=False):
+                softcap=0.0, split=True, dist_slopes=None, chunk=0, out_f32=False, dist_bias=None):
     """q fp32 [T, heads, dim] -> [T, heads, vdim] in the cache dtype (fp32 with out_f32); gate fp32 logits [T, heads]
     (one per head) or [T, heads vdim] (one per output element) or None; dist_slopes fp32 [heads]: scores are lowered by
     slope (i - j); chunk > 0: position i sees j <= i of its own chunk only.  A value cache with fewer heads than the key
-    cache: key head g reads value head g % v_heads."""
-    _cuda(q, k_cache, v_cache, sink, gate, cu_seqlens_q, context_lens, block_tables, dist_slopes)
+    cache: key head g reads value head g % v_heads.  dist_bias fp32 [heads, n]: scores gain dist_bias[h, min(i - j, n - 1)]."""
+    _cuda(q, k_cache, v_cache, sink, gate, cu_seqlens_q, context_lens, block_tables, dist_slopes, dist_bias)
     T, H, dk = q.shape
     G, dv = k_cache.shape[2], v_cache.shape[3]
     out = torch.empty(T, H, dv, dtype=torch.float32 if out_f32 else k_cache.dtype, device=q.device)
@@ -543,7 +582,7 @@ def window_attn(q, k_cache, v_cache, sink, gate, cu_seqlens_q, context_lens, blo
                                                             int(keep_first)) if split else 0
     ws = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
     opt = _attn_options(dist_slopes=dist_slopes, gate_elems=gate is not None and gate.shape[1] == H * dv and dv > 1,
-                        v_heads=v_cache.shape[2], chunk=chunk, out_f32=out_f32)
+                        v_heads=v_cache.shape[2], chunk=chunk, out_f32=out_f32, dist_bias=dist_bias)
     _lib.lib().b200_window_attn_ex(_p(out), _p(q), _p(k_cache), _p(v_cache), _p(sink), _p(gate),
                                    gate.shape[1] if gate is not None else 0, _p(cu_seqlens_q), _p(context_lens),
                                    _p(block_tables), block_tables.shape[1], context_lens.shape[0], T, H, G, dk, dv,
@@ -599,15 +638,52 @@ def attn_finish(a, gate, positions, *, heads, maps=1, lam=0.0, v_rot_freq=None, 
     return out
 
 
+NORM_KINDS = {"rms": 0, "dyntanh": 1, "layer": 2}
+
+
+def hyper_step(x, *, y=None, experts=None, mix=None, out_w=None, in_w=None, w=None, bias=None, kind="layer", alpha=1.0,
+               eps=1e-6, w_offset=0.0, rows=None, equal_streams=0, store=True, dtype=torch.float32):
+    """The step between two sublayers of hyper-connected streams.  x fp32 [S, T, D], or [T, D] with equal_streams = S (all
+    streams equal those rows).  y fp32 [T, D] or experts = (rows, slot_of_pair, top_w) of moe_experts_rows: the streams
+    become sum_s mix[s, t] x_s + out_w[t] y.  w given: the norm of sum_t in_w[t] z_t (in_w None: ones) in `dtype`, of the
+    listed `rows` only where given (then nothing is stored).  Returns (new streams [S, T, D] or None, normed rows or None)."""
+    down, slot, top_w = experts if experts is not None else (None, None, None)
+    _cuda(x, y, down, slot, top_w, mix, out_w, in_w, w, bias, rows)
+    S = equal_streams or x.shape[0]
+    T, D = x.shape[-2], x.shape[-1]
+    store = store and rows is None and (y is not None or down is not None)
+    new = torch.empty(S, T, D, dtype=torch.float32, device=x.device) if store else None
+    n = T if rows is None else rows.shape[0]
+    out = torch.empty(n, D, dtype=dtype, device=x.device) if w is not None else None
+    _lib.lib().b200_hyper_step(_p(out), _p(new), T * D, _p(x), 0 if equal_streams else T * D, _p(y), _p(down), _p(slot),
+                               _p(top_w), top_w.shape[1] if top_w is not None else 0, _p(mix), _p(out_w), _p(in_w), _p(w),
+                               _p(bias), float(alpha), NORM_KINDS[kind], float(eps), float(w_offset), _p(rows), S, n, D,
+                               _dt(dtype), _stream())
+    _lib.check()
+    return new, out
+
+
+def ff_act(up, bias, act, n=None, dtype=torch.float32):
+    """up fp32 [T, ld] -> act(up[:, :n] + bias) in `dtype`; act "relu2" or "gelu" (exact)."""
+    _cuda(up, bias)
+    T, ld = up.shape
+    n = n or ld
+    out = torch.empty(T, n, dtype=dtype, device=up.device)
+    _lib.lib().b200_ff_act(_p(out), _p(up), ld, _p(bias), {"relu2": 1, "gelu": 2}[act], T, n, _dt(dtype), _stream())
+    _lib.check()
+    return out
+
+
 def stream_norm(x, w, bias, *, kind="dyntanh", alpha=1.0, eps=1e-6, w_offset=0.0, shift_w=None, shift_state=None,
                 state_slots=None, cu_seqlens_q=None, context_lens=None, dtype=torch.float32):
-    """x fp32 [T, D] -> norm(x) in `dtype`: kind "rms" (x / rms(x) * (w_offset + w)) or "dyntanh" (tanh(alpha x) w + b).
+    """x fp32 [T, D] -> norm(x) in `dtype`: kind "rms" (x / rms(x) * (w_offset + w)), "dyntanh" (tanh(alpha x) w + b) or
+    "layer" ((x - mean) / std * (w_offset + w) + b).
     With shift_w the token shift follows: out[t] = n[t] + (n[t-1] - n[t]) * shift_w, n[t-1] from the row above or, for a
     portion's first row, from shift_state [slots, D] (zeros at position 0); shift_state is updated."""
     _cuda(x, w, bias, shift_w, shift_state, state_slots, cu_seqlens_q, context_lens)
     T, D = x.shape
     out = torch.empty(T, D, dtype=dtype, device=x.device)
-    _lib.lib().b200_stream_norm(_p(out), _p(x), _p(w), _p(bias), float(alpha), {"rms": 0, "dyntanh": 1}[kind], float(eps),
+    _lib.lib().b200_stream_norm(_p(out), _p(x), _p(w), _p(bias), float(alpha), NORM_KINDS[kind], float(eps),
                                 float(w_offset), None, _p(shift_w), _p(shift_state), _p(state_slots), _p(cu_seqlens_q),
                                 _p(context_lens), context_lens.shape[0] if context_lens is not None else 0, T, D,
                                 _dt(dtype), _stream())
@@ -616,7 +692,7 @@ def stream_norm(x, w, bias, *, kind="dyntanh", alpha=1.0, eps=1e-6, w_offset=0.0
 
 
 def depth_mix(hist, w):
-    """hist fp32 [n, ...] (contiguous), w fp32 [n] -> sum_j w[j] hist[j]."""
+    """hist fp32 [n, ...] (contiguous), w fp32 [n] (None: ones) -> sum_j w[j] hist[j]."""
     _cuda(hist, w)
     out = torch.empty_like(hist[0])
     _lib.lib().b200_depth_mix(_p(out), _p(hist), hist[0].numel(), _p(w), hist.shape[0], hist[0].numel(), _stream())
