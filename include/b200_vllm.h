@@ -703,6 +703,16 @@ void b200_runner_set_tp_fused(b200_runner*, int32_t on);
 #define B200_NORM_RMS 0
 #define B200_NORM_DYNTANH 1
 #define B200_NORM_LAYER 2
+/* What an expert does between its two products (b200_expert_act.kind).  SILU: SiLU(g) * u.  RELU2: relu(u)^2 (no gate
+ * rows).  CLAMPED: g' = min(g, limit), u' = clamp(u, -limit, limit), g' * sigmoid(alpha g') * (u' + up_add).
+ * g, u: the expert's gate and up rows.                                                                              */
+#define B200_EXPERT_SILU 0
+#define B200_EXPERT_RELU2 1
+#define B200_EXPERT_CLAMPED 2
+typedef struct b200_expert_act {
+  int32_t kind;
+  float limit, alpha, up_add;               /* CLAMPED */
+} b200_expert_act;
 
 void b200_resid_rmsnorm(void* out, const float* x, const float* w, int32_t num_tokens, int32_t width, float eps,
                         float w_offset, int32_t dt, int64_t stream);
@@ -713,6 +723,18 @@ void b200_gated_group_norm(void* out, const float* y, int32_t ldy, const float* 
 /* x fp32 [T, width] += y / sqrt(mean(y^2) + eps) * (w_offset + w): the norm after a sublayer and its residual sum */
 void b200_resid_add_rmsnorm(float* x, const float* y, const float* w, int32_t num_tokens, int32_t width, float eps,
                             float w_offset, int64_t stream);
+/* RMS norm of rows that are part of a longer row (stride ldx): out [T, n] (dtype dt) = x / sqrt(mean(x^2) + eps) * (w_offset + w) */
+void b200_rmsnorm_rows(void* out, const float* x, int32_t ldx, const float* w, int32_t num_tokens, int32_t n, float eps,
+                       float w_offset, int32_t dt, int64_t stream);
+/* out [T, n] (dtype dt) = in * sigmoid(gate); in fp32 [T, n], gate fp32 with row stride ld_gate */
+void b200_gate_rows(void* out, const float* in, const float* gate, int32_t ld_gate, int32_t num_tokens, int32_t n,
+                    int32_t dt, int64_t stream);
+/* Rotary positions in place on `heads` neighbouring heads of `dim` entries (fp32 rows with stride ld): the first rot_dims
+ * entries of every head turn by position * rot_freq[i] (f64 [rot_dims / 2]), cos and sin times rot_mag; pairs are
+ * (i, i + rot_dims / 2) when rot_half != 0, else (2i, 2i + 1).                                                      */
+void b200_rotary_rows(float* x, int32_t ld, const double* rot_freq, float rot_mag, int32_t rot_half,
+                      const int64_t* positions, int32_t num_tokens, int32_t heads, int32_t dim, int32_t rot_dims,
+                      int64_t stream);
 /* A norm of the stream with an optional token shift behind it.  n[t] = norm(x[t]) (kind B200_NORM_*; bias may be NULL);
  * with shift_w (fp32 [width]): out[t] = n[t] + (n[t-1] - n[t]) * shift_w, n[t-1] being the un-shifted norm of the
  * sequence's previous token: the row before in this step, or shift_state[slot] (fp32 [slots, width]) for the first row
@@ -728,7 +750,7 @@ void b200_stream_norm(void* out, const float* x, const float* w, const float* bi
  *   y != NULL or down != NULL:  Z_t = sum_s mix[s * streams + t] X_s + out_w[t] * y   (else Z = X)
  *   x_out != NULL: stream t is stored at x_out + t * out_stride (x_out may be x_in with the same stride)
  *   out   != NULL: out[r] = norm(sum_t in_w[t] Z_t) in dtype dt (in_w NULL: ones)
- * mix, out_w, in_w, w, bias: fp32 on the device (bias may be NULL).  rows (u32 [T], may be NULL; then x_out is NULL): row r
+ * mix, out_w, in_w, w, bias: fp32 on the device (bias may be NULL; mix NULL: the identity, out_w NULL: ones).  rows (u32 [T], may be NULL; then x_out is NULL): row r
  * of out belongs to stream row rows[r].  The sublayer's rows are y fp32 [*, width] or, where `down` is given, the weighted
  * sum of routed experts sum_j top_w[p] * down[slot_of_pair[p]], p = row * top + j (b200_moe_experts_rows).          */
 void b200_hyper_step(void* out, float* x_out, int64_t out_stride, const float* x_in, int64_t in_stride, const float* y,
@@ -853,6 +875,14 @@ void b200_latent_prep(const float* qc, int32_t ldq, void* q_plain, float* q_full
                       const float* latent_norm_w, const double* rot_freq, float rot_mag, const int64_t* positions,
                       const int64_t* slot_mapping, int32_t num_tokens, int32_t heads, int32_t dim, int32_t rot_dim,
                       int32_t rot_dims, int32_t kv_rank, float eps, int32_t dt, int64_t stream);
+/* b200_latent_prep with the queries and the raw latent row in different buffers (queries that come from a latent of their
+ * own) and a choice of rotary pairs: q fp32 [T, ldq] = heads x (dim + rot_dim), low fp32 [T, ld_low] = [latent (kv_rank) |
+ * shared rotated key (rot_dim)]; rot_half != 0: pairs (i, i + rot_dims / 2), else (2i, 2i + 1).  cache NULL: queries only. */
+void b200_latent_prep_ex(const float* q, int32_t ldq, const float* low, int32_t ld_low, void* q_plain, float* q_full,
+                         void* cache, const float* latent_norm_w, const double* rot_freq, float rot_mag,
+                         int32_t rot_half, const int64_t* positions, const int64_t* slot_mapping, int32_t num_tokens,
+                         int32_t heads, int32_t dim, int32_t rot_dim, int32_t rot_dims, int32_t kv_rank, float eps,
+                         int32_t dt, int64_t stream);
 /* out [T, heads, kv_rank] (dtype dt) = softmax-weighted sum of cached latents; sink fp32 [heads] or NULL;
  * window <= 0: full causal context.  cache [num_blocks, 64, kv_rank + rot_dim].  workspace (may be NULL):
  * b200_latent_attn_workspace_bytes() bytes; with it, steps of few token rows split each row's keys over several
@@ -923,7 +953,8 @@ void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, cons
                          int32_t width, int32_t ff, int32_t act, int32_t accumulate, const void* ident,
                          int32_t ident_f32, int32_t dt, void* workspace, int64_t stream);
 
-/* Router scores and weights beyond b200_moe_route_ex.  score 0: softmax over all outputs, 1: the sigmoid of every logit;
+/* Router scores and weights beyond b200_moe_route_ex.  score 0: softmax over all outputs, 1: the sigmoid of every logit,
+ * 2: the logit + bias itself, the weights being a softmax over the chosen ones only;
  * group_top: a group's score is the sum of its group_top (1 or 2) largest choice scores; renorm != 0: the chosen weights
  * are divided by their sum + 1e-20 (before `scale`).                                                                */
 void b200_moe_route_full(const float* logits, const float* bias, int32_t num_tokens, int32_t experts, int32_t top,
@@ -935,6 +966,15 @@ void b200_moe_experts_rows(const void* h, const int32_t* top_idx, const void* w_
                            int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff, int32_t act,
                            int32_t dt, void* workspace, const float** down, const int32_t** slot_of_pair,
                            int64_t stream);
+/* b200_moe_experts_ex and b200_moe_experts_rows with any expert activation (act: host) */
+void b200_moe_experts_act(float* out, const void* h, const int32_t* top_idx, const float* top_w, const void* w_up,
+                          const void* w_down, int32_t num_tokens, int32_t experts, int32_t identity, int32_t top,
+                          int32_t width, int32_t ff, const b200_expert_act* act, int32_t accumulate, const void* ident,
+                          int32_t ident_f32, int32_t dt, void* workspace, int64_t stream);
+void b200_moe_experts_rows_act(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down,
+                               int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff,
+                               const b200_expert_act* act, int32_t dt, void* workspace, const float** down,
+                               const int32_t** slot_of_pair, int64_t stream);
 
 typedef struct b200_hybrid_config {
   int32_t width, vocab, num_layers;
@@ -991,7 +1031,7 @@ typedef struct b200_hybrid_layer {
   int32_t gated;                            /* window attention: != 0: per-head sigmoid output gate, logits last in w_in */
   void* v_cache;                            /* window attention: kv_cache holds K, v_cache V */
   /* ---- POSTNORM layers, attention with a distance bias, shared latent caches, routers with groups
-   * gated (both attentions): 1 = one gate logit per head, 2 = one per output element (window attention only); the
+   * gated (both attentions): 1 = one gate logit per head, 2 = one per output element (heads x vdim); the
    * logits are the last rows of w_in.  w_in of a latent attention with shared_cache: the queries (and gate) only. */
   int32_t head_norm, v_from_k;              /* window attention: see b200_attn_options */
   int32_t q_temp_every;
@@ -999,7 +1039,7 @@ typedef struct b200_hybrid_layer {
   const void* dist_slopes;                  /* fp32 [heads] or NULL */
   int32_t shared_cache;                     /* latent attention: != 0: no latent projection of its own; kv_cache is
                                                another (earlier) layer's cache, which this layer only reads */
-  int32_t expert_act, shared_act;           /* 0: SiLU(gate) * up ([gate | up] rows); 1: relu(up)^2 (up rows only);
+  int32_t expert_act, shared_act;           /* expert_act: B200_EXPERT_*; shared_act 0: SiLU(gate) * up ([gate | up] rows); 1: relu(up)^2 (up rows only);
                                                2 (shared_act): the exact GELU of up (up rows only) */
   int32_t identity_experts;                 /* router outputs experts .. experts + identity_experts - 1 return the input */
   int32_t route_groups, route_keep;         /* see b200_moe_route_ex (0: no groups) */
@@ -1015,7 +1055,7 @@ typedef struct b200_hybrid_layer {
   void* shift_state;                        /* fp32 [slots, width], caller-owned */
   const void* depth_w;                      /* fp32 [layer + 2] or NULL: the layer's result X_(layer+1) is kept, and what
                                                goes on is sum_j depth_w[j] X_j, X_0 being the embedding output */
-  float ff_scale;                           /* PRENORM: the feed-forward's output is multiplied by it */
+  float ff_scale;                           /* PRENORM: the feed-forward's output is multiplied by it (experts and shared part) */
   const void *ff_up_bias, *ff_down_bias;    /* fp32 [shared_ff], [width] or NULL: biases of a squared-ReLU dense feed-forward */
   /* window attention (see b200_attn_options).  score_maps == 2: differential attention; w_in holds
    * [q: maps x heads x dim | k: maps x kv_heads x dim | v: kv_heads x vdim | gate], the maps one after the other, the
@@ -1042,6 +1082,14 @@ typedef struct b200_hybrid_layer {
                                                layers have the same kv_heads x vdim                                   */
   float v_mix;
   int32_t route_score, route_group_top, route_renorm;   /* see b200_moe_route_full (route_group_top 0 reads as 1) */
+  /* ---- latent queries, rotated decay attention, clamped experts
+   * latent attention: q_rank > 0: the queries go through a latent: w_in = [query latent: q_rank | latent: kv_rank | rotated
+   * key: rot_dim | gate logits], the query latent is RMS-normed (q_norm_w fp32 [q_rank], no offset) and w_uq (dtype dt,
+   * [heads x (dim + rot_dim), q_rank]) makes the queries.  rot_half (both attentions and decay attention) chooses the pairs.
+   * decay attention: rot_dims > 0: the first rot_dims entries of every q and k head are rotated by their position.      */
+  int32_t q_rank;
+  const void* w_uq;
+  float expert_limit, expert_alpha, expert_up_add;      /* expert_act B200_EXPERT_CLAMPED, see b200_expert_act */
 } b200_hybrid_layer;
 
 typedef struct b200_hybrid b200_hybrid;

@@ -92,7 +92,14 @@ class HybridLayer(C.Structure):
                [("chan_rank", c_i32), ("gate_rank", c_i32), ("w_gate2", c_vp)] + \
                [(n, c_vp) for n in ("hc_in", "hc_mix", "hc_out", "ff_hc_in", "ff_hc_mix", "ff_hc_out", "dist_bias")] + \
                [("dist_n", c_i32), ("v_mix_role", c_i32), ("v_mix", c_f32)] + \
-               [(n, c_i32) for n in ("route_score", "route_group_top", "route_renorm")]
+               [(n, c_i32) for n in ("route_score", "route_group_top", "route_renorm", "q_rank")] + [("w_uq", c_vp)] + \
+               [(n, c_f32) for n in ("expert_limit", "expert_alpha", "expert_up_add")]
+
+
+class ExpertAct(C.Structure):
+    """b200_expert_act (include/b200_vllm.h)."""
+
+    _fields_ = [("kind", c_i32)] + [(n, c_f32) for n in ("limit", "alpha", "up_add")]
 
 
 class KvCachePlan(C.Structure):
@@ -288,6 +295,13 @@ _SIGS = {
     "b200_moe_experts_rows": (None, [c_vp] * 4 + [c_i32] * 7 + [c_vp, c_vp, c_vp, c_i64]),
     "b200_moe_experts_ex": (None, [c_vp] * 6 + [c_i32] * 8 + [c_vp, c_i32, c_i32, c_vp, c_i64]),
     "b200_moe_experts": (None, [c_vp] * 6 + [c_i32] * 6 + [c_vp, c_i64]),
+    "b200_moe_experts_act": (None, [c_vp] * 6 + [c_i32] * 6 + [C.POINTER(ExpertAct), c_i32, c_vp, c_i32, c_i32, c_vp, c_i64]),
+    "b200_moe_experts_rows_act": (None, [c_vp] * 4 + [c_i32] * 5 + [C.POINTER(ExpertAct), c_i32] + [c_vp] * 3 + [c_i64]),
+    "b200_rmsnorm_rows": (None, [c_vp, c_vp, c_i32, c_vp, c_i32, c_i32, c_f32, c_f32, c_i32, c_i64]),
+    "b200_gate_rows": (None, [c_vp] * 3 + [c_i32] * 4 + [c_i64]),
+    "b200_rotary_rows": (None, [c_vp, c_i32, c_vp, c_f32, c_i32, c_vp] + [c_i32] * 4 + [c_i64]),
+    "b200_latent_prep_ex": (None, [c_vp, c_i32, c_vp, c_i32] + [c_vp] * 5 + [c_f32, c_i32, c_vp, c_vp] + [c_i32] * 6 +
+                            [c_f32, c_i32, c_i64]),
     "b200_hybrid_new": (c_vp, [C.POINTER(HybridConfig)]),
     "b200_hybrid_free": (None, [c_vp]),
     "b200_hybrid_set_layer": (None, [c_vp, c_i32, C.POINTER(HybridLayer)]),

@@ -6,9 +6,10 @@
 //   h = norm(x)                                                    resid_rmsnorm        (fp32 in, operand dtype out)
 //   latent attention:  [q | latent | k_rot] = h W_in^T             library GEMM (fp32 out)
 //                      norm + rotary + cache write + query split   latent_prep
+//                      (latent queries: [q_low | latent | k_rot] = h W_in^T ; rmsnorm_rows ; q = . W_uq^T before it)
 //                      q_abs[h] = q_plain[h] W_uk[h]               batched library GEMM into q_full
 //                      latent_attn (window, sink)                  -> attention-weighted latents
-//                      v[h] = lat[h] W_uv[h]^T ; x += v W_o^T      batched GEMM, cast, GEMM with beta = 1
+//                      v[h] = lat[h] W_uv[h]^T ; x += v W_o^T      batched GEMM, cast (times the element gate), GEMM with beta = 1
 //   delta rule:        [q | k | v | b | a | gate] = h W_in^T ; short_conv_silu on q | k | v ; delta_rule ;
 //                      gated_group_norm (gate after the norm) ; x += . W_o^T
 //   SSD:               [z | x | B | C | dt] = h W_in^T ; short_conv_silu on x | B | C ; ssd_scan ;
@@ -16,8 +17,8 @@
 //   window attention:  [q | k | v | gate] = h W_in^T ; window_attn_prep (biases, whole-projection q / k norms, rotary,
 //                      K / V cache write) ; window_attn (window + kept first tokens, capped scores, sink, gate) ;
 //                      dst (+)= scale . W_o^T (+ bias)
-//   decay attention:   [q | k | v | gate | low] = h W_in^T ; lowrank_decay (per-channel decays) ; decay_attn ;
-//                      gated_group_norm ; dst (+)= scale . W_o^T
+//   decay attention:   [q | k | v | gate | low] = h W_in^T ; rotary_rows on q | k ; lowrank_decay (per-channel decays) ;
+//                      decay_attn ; gated_group_norm ; dst (+)= scale . W_o^T
 //   experts:           router GEMM (fp32 out) -> moe_route -> sort -> grouped gate|up (SiLU * mul) -> grouped down ->
 //                      combine into x ; shared expert: GEMM, silu_mul, GEMM with beta = 1 into x
 // The residual add of every branch is the beta = 1 accumulation of its last matrix product (or the combine kernel).
@@ -29,7 +30,8 @@
 // feed-forward being the routed experts (plus their shared expert) or the dense gated one.
 // Pre-norm layer (each sublayer behind its own norm, added times a factor): h = norm(x) -- RMS or dynamic tanh, with the
 // token shift h[t] += (h[t-1] - h[t]) * shift where the layer has one (stream_norm) --, x += out_scale * mixer(h);
-// h = ff_norm(x), x += ff_scale * ff(h).  With depth weights the layers' results X_0 (embedding) .. X_L are kept side by
+// h = ff_norm(x), x += ff_scale * ff(h).  Routed experts leave their rows unsummed where a norm follows at once: hyper_step
+// (with one stream) weighs them, updates x and writes the next norm in one pass.  With depth weights the layers' results X_0 (embedding) .. X_L are kept side by
 // side, layer i works in place on slot i + 1 (which starts as its input), and depth_mix writes
 // sum_j depth_w[j] X_j into slot i + 2 (the stream for the last layer), which is the next layer's input.
 // Hyper-connected layer (pre-norm sublayers over S residual streams): hyper_step = the update that closes the previous
@@ -134,7 +136,8 @@ static bool graphs_enabled() {
 static int in_rows(const b200_hybrid_layer& l) {
   switch (l.mixer) {
     case B200_MIXER_LATENT_ATTN:
-      return l.heads * (l.dim + l.rot_dim) + (l.shared_cache ? 0 : l.kv_rank + l.rot_dim) + (l.gated ? l.heads : 0);
+      return (l.q_rank > 0 ? l.q_rank : l.heads * (l.dim + l.rot_dim)) + (l.shared_cache ? 0 : l.kv_rank + l.rot_dim) +
+             (l.gated == 2 ? l.heads * l.vdim : (l.gated ? l.heads : 0));
     case B200_MIXER_DELTA_RULE:
       if (l.chan_rank > 0) return 2 * l.kv_heads * l.dim + l.heads * l.vdim + l.heads + l.chan_rank + l.gate_rank;
       return 2 * l.kv_heads * l.dim + 2 * l.heads * l.vdim + 2 * l.heads;
@@ -183,7 +186,8 @@ static int64_t carve(b200_hybrid* r, uint8_t* base) {
     } else if (l.mixer == B200_MIXER_LATENT_ATTN) {
       aux_n = std::max<size_t>(aux_n, static_cast<size_t>(l.heads) * std::max(l.kv_rank + l.rot_dim, l.vdim));
       opa_n = std::max<size_t>(opa_n, static_cast<size_t>(l.heads) * std::max(l.dim, l.vdim));
-      lat_n = std::max<size_t>(lat_n, static_cast<size_t>(l.heads) * l.kv_rank);
+      lat_n = std::max<size_t>(lat_n, std::max<size_t>(static_cast<size_t>(l.heads) * l.kv_rank, l.q_rank));
+      if (l.q_rank > 0) conv_n = std::max<size_t>(conv_n, static_cast<size_t>(l.heads) * (l.dim + l.rot_dim));
       for (size_t rows = 1; rows <= r->attn_ws_rows; ++rows)
         attn_bytes = std::max(attn_bytes, latent_attn_workspace_bytes(static_cast<int>(rows), l.heads, l.kv_rank, l.window));
     } else {
@@ -279,7 +283,8 @@ static bool mixer_ok(const b200_hybrid_layer* l) {
            l->v_mix_role >= 0 && l->v_mix_role <= 2 && (l->v_mix_role == 0 || !l->shared_cache);
   if (l->mixer == B200_MIXER_DECAY_ATTN)
     return ok && l->dim > 0 && l->dim <= 256 && l->rec_state && l->norm_groups > 0 &&
-           (l->heads * l->vdim) % l->norm_groups == 0 && (l->out_norm_period == 0 || l->out_norm_w) &&
+           (l->heads * l->vdim) % l->norm_groups == 0 && (l->out_norm_period == 0 || l->out_norm_w) && l->rot_dims >= 0 &&
+           l->rot_dims % 2 == 0 && l->rot_dims <= l->dim && (l->rot_dims == 0 || l->rot_freq) &&
            (l->decay_rank > 0 ? (l->w_decay2 && l->decay_tau > 0.f) : l->head_decay != nullptr);
   return false;
 }
@@ -314,7 +319,7 @@ void b200_hybrid_set_layer(b200_hybrid* r, int32_t layer, const b200_hybrid_laye
     ok = ok && l->hc_in && l->hc_mix && l->hc_out && !l->shift_w && !l->depth_w && l->out_scale == 1.f && l->ff_scale == 1.f &&
          (!with_ff || (l->ff_norm_w && l->ff_hc_in && l->ff_hc_mix && l->ff_hc_out));
   if (l->layout == B200_LAYOUT_PRENORM)
-    ok = ok && ((l->shared_ff == 0 && l->experts == 0) || l->ff_norm_w) && (l->experts == 0 || l->ff_scale == 1.f);
+    ok = ok && ((l->shared_ff == 0 && l->experts == 0) || l->ff_norm_w);
   ok = ok && l->norm_kind >= B200_NORM_RMS && l->norm_kind <= B200_NORM_LAYER && (!l->shift_w || l->shift_state) &&
        ((!l->shift_w && !l->depth_w && !l->ff_up_bias && !l->ff_down_bias && l->norm_kind == B200_NORM_RMS) ||
         l->layout == B200_LAYOUT_PRENORM || hyper) &&
@@ -324,7 +329,8 @@ void b200_hybrid_set_layer(b200_hybrid* r, int32_t layer, const b200_hybrid_laye
   else if (l->mixer == B200_MIXER_LATENT_ATTN)
     ok = ok && l->kv_rank > 0 && l->w_uk && l->w_uv && (l->shared_cache || l->latent_norm_w) && l->kv_cache &&
          l->rot_dims % 2 == 0 && l->rot_dims <= l->rot_dim && (l->rot_dims == 0 || l->rot_freq) &&
-         (l->gated == 0 || l->gated == 1) && (!l->shared_cache || l->rot_dim == 0);
+         l->gated >= 0 && l->gated <= 2 && (!l->shared_cache || l->rot_dim == 0) && l->q_rank >= 0 &&
+         (l->q_rank == 0 || (l->w_uq && l->q_norm_w));
   else if (l->mixer == B200_MIXER_DELTA_RULE)
     ok = ok && l->kv_heads > 0 && l->heads % l->kv_heads == 0 && l->dim > 0 && l->conv_taps >= 1 && l->conv_w &&
          l->conv_state && l->rec_state && l->a_log && l->dt_bias && l->out_norm_w && l->chan_rank >= 0 &&
@@ -338,8 +344,8 @@ void b200_hybrid_set_layer(b200_hybrid* r, int32_t layer, const b200_hybrid_laye
   if (l->experts > 0) {
     const int all = l->experts + l->identity_experts;
     ok = ok && l->identity_experts >= 0 && l->top > 0 && l->top <= all && l->expert_ff > 0 && l->w_router &&
-         l->w_gate_up && l->w_down && (l->expert_act == 0 || l->expert_act == 1) && l->route_groups >= 0 &&
-         (l->route_score == 0 || l->route_score == 1) && l->route_group_top >= 0 && l->route_group_top <= 2 &&
+         l->w_gate_up && l->w_down && l->expert_act >= B200_EXPERT_SILU && l->expert_act <= B200_EXPERT_CLAMPED &&
+         l->expert_limit >= 0.f && l->route_groups >= 0 && l->route_score >= 0 && l->route_score <= 2 && l->route_group_top >= 0 && l->route_group_top <= 2 &&
          (l->route_groups == 0 || (all % l->route_groups == 0 && l->route_keep >= 1 && l->route_keep <= l->route_groups &&
                                    l->top <= all / l->route_groups * l->route_keep));
   } else {
@@ -425,25 +431,38 @@ static void mixer_latent(b200_hybrid* r, const b200_hybrid_layer& l, const int64
   const b200_hybrid_config& c = r->cfg;
   const int H = l.heads, R = l.kv_rank + l.rot_dim, n_in = in_rows(l);
   gemm_f32out(r->hin, c.width, 0, l.w_in, c.width, 0, r->proj, n_in, 0, T, n_in, c.width, 1, 0.f, 0, c.dt, st);
+  const float* q = r->proj;
+  int ld_q = n_in, n_q = H * (l.dim + l.rot_dim);
+  const float* low = r->proj + (l.q_rank > 0 ? l.q_rank : n_q);
+  if (l.q_rank > 0) {            // queries from a latent of their own (its normed rows borrow the buffer of the result)
+    launch_resid_rmsnorm(r->lat, r->proj, (const float*)l.q_norm_w, T, l.q_rank, c.norm_eps, 0.f, nullptr, c.dt, st, n_in);
+    gemm_f32out(r->lat, l.q_rank, 0, l.w_uq, l.q_rank, 0, r->conv, n_q, 0, T, n_q, l.q_rank, 1, 0.f, 0, c.dt, st);
+    q = r->conv;
+    ld_q = n_q;
+  }
   // a layer that shares another layer's cache brings queries only: nothing is normed or written
-  launch_latent_prep(r->proj, n_in, r->opa, r->aux, l.shared_cache ? nullptr : l.kv_cache, (const float*)l.latent_norm_w,
-                     l.rot_freq, l.rot_mag, positions, slots, T, H, l.dim, l.rot_dim, l.rot_dims, l.kv_rank, c.norm_eps,
-                     c.dt, st);
+  launch_latent_prep(q, ld_q, low, n_in, r->opa, r->aux, l.shared_cache ? nullptr : l.kv_cache,
+                     (const float*)l.latent_norm_w, l.rot_freq, l.rot_mag, l.rot_half, positions, slots, T, H, l.dim,
+                     l.rot_dim, l.rot_dims, l.kv_rank, c.norm_eps, c.dt, st);
   // q_abs[t, h, :] = q_plain[t, h, :] W_uk[h]  (W_uk[h] is [dim, kv_rank], i.e. stored [K, N])
   if (l.dim > 0)
     gemm_f32out(r->opa, H * l.dim, l.dim, l.w_uk, l.kv_rank, static_cast<long long>(l.dim) * l.kv_rank, r->aux, H * R, R,
                 T, l.kv_rank, l.dim, H, 0.f, 1, c.dt, st);
   else
     cudaMemsetAsync(r->aux, 0, static_cast<size_t>(T) * H * R * 4, st);   // (rotated parts are rewritten by prep; dim == 0 is rejected upstream)
-  const float* gate = l.gated ? r->proj + (n_in - H) : nullptr;          // the gate logits close the projection row
-  launch_latent_attn(r->lat, r->aux, l.kv_cache, (const float*)l.sink, gate, n_in, cu, ctx, bt, max_blocks, B, T, H,
+  // the gate logits close the projection row; one per head joins the attention, one per element waits for the values
+  const float* gate = l.gated ? r->proj + (n_in - (l.gated == 2 ? H * l.vdim : H)) : nullptr;
+  launch_latent_attn(r->lat, r->aux, l.kv_cache, (const float*)l.sink, l.gated == 1 ? gate : nullptr, n_in, cu, ctx, bt, max_blocks, B, T, H,
                      l.kv_rank, l.rot_dim, l.window, l.scale, c.dt,
                      static_cast<size_t>(T) <= r->attn_ws_rows ? r->attn_ws : nullptr, st);
   // v[t, h, :] = lat[t, h, :] W_uv[h]^T  (W_uv[h] is [vdim, kv_rank])
   gemm_f32out(r->lat, H * l.kv_rank, l.kv_rank, l.w_uv, l.kv_rank, static_cast<long long>(l.vdim) * l.kv_rank, r->aux,
               H * l.vdim, l.vdim, T, l.vdim, l.kv_rank, H, 0.f, 0, c.dt, st);
   const void* o_in = r->aux;
-  if (!c.dt) {
+  if (l.gated == 2) {
+    launch_gate_rows(r->opa, r->aux, gate, n_in, T, H * l.vdim, c.dt, st);
+    o_in = r->opa;
+  } else if (!c.dt) {
     launch_cast_rows(r->opa, r->aux, H * l.vdim, T, H * l.vdim, 0, st);
     o_in = r->opa;
   }
@@ -554,7 +573,7 @@ static void mixer_window(b200_hybrid* r, const b200_hybrid_layer& l, const int64
   if (l.o_bias) launch_bias_rows(dst, (const float*)l.o_bias, alpha, T, c.width, st);
 }
 
-static void mixer_decay(b200_hybrid* r, const b200_hybrid_layer& l, const uint32_t* cu, const uint32_t* ctx,
+static void mixer_decay(b200_hybrid* r, const b200_hybrid_layer& l, const int64_t* positions, const uint32_t* cu, const uint32_t* ctx,
                         const int32_t* state_slots, int B, int T, float* dst, float alpha, float beta, cudaStream_t st) {
   const b200_hybrid_config& c = r->cfg;
   const int H = l.heads, nk = H * l.dim, nv = H * l.vdim, n_in = in_rows(l);
@@ -564,6 +583,8 @@ static void mixer_decay(b200_hybrid* r, const b200_hybrid_layer& l, const uint32
   const float* v = k + nk;
   const float* gate = v + nv;
   const float* chan = nullptr;
+  if (l.rot_dims > 0)            // q and k heads lie side by side and turn in place
+    launch_rotary_rows(r->proj, n_in, l.rot_freq, l.rot_mag, l.rot_half, positions, T, 2 * H, l.dim, l.rot_dims, st);
   if (l.decay_rank > 0) {
     launch_lowrank_decay(r->conv, gate + nv, n_in, (const float*)l.w_decay2, (const float*)l.decay_bias, l.decay_tau,
                          nullptr, 1, T, nk, l.decay_rank, st);
@@ -590,7 +611,7 @@ static void run_mixer(b200_hybrid* r, const b200_hybrid_layer& l, const int64_t*
     case B200_MIXER_WINDOW_ATTN:
       mixer_window(r, l, positions, slot_mapping, cu, ctx, block_tables, max_blocks, B, T, dst, alpha, beta, st);
       break;
-    case B200_MIXER_DECAY_ATTN: mixer_decay(r, l, cu, ctx, state_slots, B, T, dst, alpha, beta, st); break;
+    case B200_MIXER_DECAY_ATTN: mixer_decay(r, l, positions, cu, ctx, state_slots, B, T, dst, alpha, beta, st); break;
     default: mixer_ssd(r, l, cu, ctx, state_slots, B, T, dst, alpha, beta, st); break;
   }
 }
@@ -605,26 +626,31 @@ static void dense_ffn(b200_hybrid* r, const b200_hybrid_layer& l, int T, cudaStr
               0, c.dt, st);
 }
 
-// the router of a layer: logits, choice and weights of every token
-static void route_tokens(b200_hybrid* r, const b200_hybrid_layer& l, int T, cudaStream_t st) {
+static b200_expert_act expert_act(const b200_hybrid_layer& l) {
+  return b200_expert_act{l.expert_act, l.expert_limit, l.expert_alpha, l.expert_up_add};
+}
+
+// the router of a layer: logits, choice and weights (times `scale`) of every token
+static void route_tokens(b200_hybrid* r, const b200_hybrid_layer& l, int T, cudaStream_t st, float scale = 1.f) {
   const b200_hybrid_config& c = r->cfg;
   const int all = l.experts + l.identity_experts;
   gemm_f32out(r->hin, c.width, 0, l.w_router, c.width, 0, r->rlog, all, 0, T, all, c.width, 1, 0.f, 0, c.dt, st);
   launch_moe_route(r->rlog, (const float*)l.route_bias, T, all, l.top, l.route_groups, l.route_keep, l.route_score,
-                   l.route_group_top, l.route_renorm, l.route_scale, r->top_idx, r->top_w, st);
+                   l.route_group_top, l.route_renorm, l.route_scale * scale, r->top_idx, r->top_w, st);
 }
 
 // routed experts and their shared expert: dst = (accumulate ? dst : 0) + experts(h) + shared(h).  `ident` / `ident_f32`:
 // the rows that identity experts return (the sublayer's input before any rounding, where the layer has it in fp32).
-// `scale` multiplies the shared / dense part (routed experts take none).
+// `scale` multiplies the result.
 static void feed_forward(b200_hybrid* r, const b200_hybrid_layer& l, int T, float* dst, bool accumulate, const void* ident,
                          int ident_f32, cudaStream_t st, float scale = 1.f) {
   const b200_hybrid_config& c = r->cfg;
   if (l.experts > 0) {
-    route_tokens(r, l, T, st);
-    b200_moe_experts_ex(dst, r->hin, r->top_idx, r->top_w, l.w_gate_up, l.w_down, T, l.experts, l.identity_experts, l.top,
-                        c.width, l.expert_ff, l.expert_act, accumulate ? 1 : 0, ident, ident_f32, c.dt, r->moe_ws,
-                        reinterpret_cast<int64_t>(st));
+    const b200_expert_act act = expert_act(l);
+    route_tokens(r, l, T, st, scale);
+    b200_moe_experts_act(dst, r->hin, r->top_idx, r->top_w, l.w_gate_up, l.w_down, T, l.experts, l.identity_experts, l.top,
+                         c.width, l.expert_ff, &act, accumulate ? 1 : 0, ident, ident_f32, c.dt, r->moe_ws,
+                         reinterpret_cast<int64_t>(st));
     accumulate = true;
   }
   if (l.shared_ff > 0) {
@@ -688,6 +714,21 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
       pend = {};
     }
   };
+  // routed experts whose rows are summed by the next hyper_step
+  auto expert_rows = [&](const b200_hybrid_layer& l, float scale) {
+    const b200_expert_act act = expert_act(l);
+    route_tokens(r, l, T, st, scale);
+    b200_moe_experts_rows_act(r->hin, r->top_idx, l.w_gate_up, l.w_down, T, l.experts, l.top, c.width, l.expert_ff, &act,
+                              c.dt, r->moe_ws, &pend.down, &pend.slot_of_pair, stream);
+    pend.top = l.top;
+  };
+  // one stream: x += the pending experts (stored unless only `rows` are wanted), out = norm(x)
+  auto settle = [&](void* out, const void* w, const void* b, float alpha, int kind, const uint32_t* rows, int n) {
+    launch_hyper_step(out, rows ? nullptr : r->x, 0, r->x, 0, nullptr, pend.down, pend.slot_of_pair, r->top_w, pend.top, nullptr,
+                      nullptr, nullptr, (const float*)w, (const float*)b, alpha, kind, c.norm_eps, c.norm_weight_offset, rows,
+                      1, n, c.width, c.dt, st);
+    pend = {};
+  };
   for (int i = 0; i < c.num_layers; ++i) {
     const b200_hybrid_layer& l = r->layers[i];
     const b200_hybrid_layer& side = r->sides[i];
@@ -735,11 +776,8 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
               l.norm_kind, nullptr, T);
         pend = {(const float*)l.ff_hc_mix, (const float*)l.ff_hc_out, r->y, nullptr, nullptr, 0};
         if (l.experts > 0 && l.shared_ff == 0 && l.identity_experts == 0) {      // the next hyper_step sums the experts' rows
-          route_tokens(r, l, T, st);
-          b200_moe_experts_rows(r->hin, r->top_idx, l.w_gate_up, l.w_down, T, l.experts, l.top, c.width, l.expert_ff,
-                                l.expert_act, c.dt, r->moe_ws, &pend.down, &pend.slot_of_pair, stream);
+          expert_rows(l, 1.f);
           pend.y = nullptr;
-          pend.top = l.top;
         } else {
           feed_forward(r, l, T, r->y, false, r->h, 0, st);
         }
@@ -752,9 +790,12 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
       continue;
     }
     if (l.layout == B200_LAYOUT_PRENORM) {
-      launch_stream_norm(r->h, r->x, (const float*)l.norm_w, (const float*)l.norm_b, l.norm_alpha, l.norm_kind, c.norm_eps,
-                         c.norm_weight_offset, nullptr, (const float*)l.shift_w, (float*)l.shift_state, state_slots, cu,
-                         ctx, B, T, c.width, c.dt, st);
+      if (pend.down)
+        settle(r->h, l.norm_w, l.norm_b, l.norm_alpha, l.norm_kind, nullptr, T);
+      else
+        launch_stream_norm(r->h, r->x, (const float*)l.norm_w, (const float*)l.norm_b, l.norm_alpha, l.norm_kind, c.norm_eps,
+                           c.norm_weight_offset, nullptr, (const float*)l.shift_w, (float*)l.shift_state, state_slots, cu,
+                           ctx, B, T, c.width, c.dt, st);
       run_mixer(r, l, positions, slot_mapping, cu, ctx, block_tables, state_slots, max_blocks, B, T, r->x, l.out_scale,
                 1.f, st);
       if (side.heads > 0)
@@ -764,7 +805,13 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
         launch_stream_norm(r->h, r->x, (const float*)l.ff_norm_w, (const float*)l.ff_norm_b, l.ff_norm_alpha, l.norm_kind,
                            c.norm_eps, c.norm_weight_offset, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, 0, T,
                            c.width, c.dt, st);
-        feed_forward(r, l, T, r->x, true, r->h, 0, st, l.ff_scale);
+        // the norm that follows takes over the sum of the experts, if there is nothing in between
+        const b200_hybrid_layer* next = i + 1 < c.num_layers ? &r->layers[i + 1] : nullptr;
+        if (l.experts > 0 && l.shared_ff == 0 && l.identity_experts == 0 && !r->hist &&
+            (!next || (next->layout == B200_LAYOUT_PRENORM && !next->shift_w)))
+          expert_rows(l, l.ff_scale);
+        else
+          feed_forward(r, l, T, r->x, true, r->h, 0, st, l.ff_scale);
       }
       if (r->hist) {
         // what goes on: the weighted sum of the results so far, or (a layer without weights) this layer's result
@@ -773,9 +820,11 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
         else cudaMemcpyAsync(next, r->x, xbytes, cudaMemcpyDeviceToDevice, st);
         r->x = next;
       }
-      if (r->trace)
+      if (r->trace) {
+        if (pend.down) settle(nullptr, nullptr, nullptr, 1.f, l.norm_kind, nullptr, T);
         cudaMemcpyAsync(r->trace + static_cast<size_t>(i) * c.max_tokens * c.width, r->x, xbytes, cudaMemcpyDeviceToDevice,
                         st);
+      }
       continue;
     }
     launch_resid_rmsnorm(r->h, r->x, (const float*)l.norm_w, T, c.width, c.norm_eps, c.norm_weight_offset, nullptr,
@@ -811,6 +860,8 @@ void b200_hybrid_step(b200_hybrid* r, const uint32_t* input_ids, const int64_t* 
     if (c.streams > 0)
       hyper(r->hr, false, nullptr, (const float*)r->final_norm, (const float*)r->final_norm_b, r->final_norm_alpha,
             c.final_norm_kind, out_rows, num_out);
+    else if (pend.down)
+      settle(r->hr, r->final_norm, r->final_norm_b, r->final_norm_alpha, c.final_norm_kind, out_rows, num_out);
     else if (c.final_norm_kind == B200_NORM_RMS)
       launch_resid_rmsnorm(r->hr, r->x, (const float*)r->final_norm, num_out, c.width, c.norm_eps, c.norm_weight_offset,
                            out_rows, c.dt, st);

@@ -19,8 +19,10 @@
 //
 // latent_prep_kernel: from the fused projection row [q (H x (dim + rot_dim)) | c_raw (kv_rank) | k_rot_raw (rot_dim)]
 // (fp32) it RMS-norms the latent (plain weight), rotates the first rot_dims entries of every head's rotated query
-// part and of the shared key part as interleaved pairs (2i, 2i+1) by the angle position * freq[i] (angles in double,
-// cos / sin scaled by rot_mag), writes the cache row at the token's slot, and splits the queries.
+// part and of the shared key part, as interleaved pairs (2i, 2i+1) or as the two halves (i, i + rot_dims / 2), by the
+// angle position * freq[i] (angles in double, cos / sin scaled by rot_mag), writes the cache row at the token's slot, and
+// splits the queries.  Queries that come from a latent of their own (a second matrix product) lie in another buffer than
+// the row with c_raw and k_rot_raw.
 #include "../../include/b200_vllm.h"
 #include <algorithm>
 #include <cstdlib>
@@ -31,10 +33,11 @@ namespace b200 {
 using namespace seqmix;
 
 template <typename T>
-__global__ void latent_prep_kernel(const float* __restrict__ qc, int ldq, T* __restrict__ q_plain,
+__global__ void latent_prep_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ low, int ld_low,
+                                   T* __restrict__ q_plain,
                                    float* __restrict__ q_full, T* __restrict__ cache,
                                    const float* __restrict__ latent_norm_w, const double* __restrict__ rot_freq,
-                                   float rot_mag, const int64_t* __restrict__ positions,
+                                   float rot_mag, int rot_half, const int64_t* __restrict__ positions,
                                    const int64_t* __restrict__ slots, int heads, int dim, int rot_dim, int rot_dims,
                                    int kv_rank, float eps) {
   extern __shared__ float sm[];          // cos[rot_dims/2] | sin[rot_dims/2] | red[33]
@@ -43,9 +46,9 @@ __global__ void latent_prep_kernel(const float* __restrict__ qc, int ldq, T* __r
   float* sn = sm + half;
   float* red = sm + 2 * half;
   const int t = blockIdx.x;
-  const float* row = qc + static_cast<size_t>(t) * ldq;
-  const bool own_latent = cache != nullptr;            // otherwise the row holds the queries only
-  const float* craw = row + static_cast<size_t>(heads) * (dim + rot_dim);
+  const float* row = q + static_cast<size_t>(t) * ldq;
+  const bool own_latent = cache != nullptr;            // otherwise there are queries only
+  const float* craw = low + static_cast<size_t>(t) * ld_low;
   const float* kraw = craw + kv_rank;
   const double pos = static_cast<double>(positions[t]);
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -59,20 +62,20 @@ __global__ void latent_prep_kernel(const float* __restrict__ qc, int ldq, T* __r
     for (int d = threadIdx.x; d < kv_rank; d += blockDim.x) ss += craw[d] * craw[d];
   ss = block_sum(ss, red);           // also orders the cos / sin writes before their use
   const float inv = 1.f / sqrtf(ss / static_cast<float>(kv_rank) + eps);
+  // entry d of a rotated part
+  auto turned = [&](const float* raw, int d) {
+    if (d >= rot_dims) return raw[d];
+    const bool second = rot_half ? d >= half : (d & 1) != 0;
+    const int i = rot_half ? (second ? d - half : d) : d >> 1;
+    const float a = raw[rot_half ? i : 2 * i], b = raw[rot_half ? i + half : 2 * i + 1];
+    return second ? b * cs[i] + a * sn[i] : a * cs[i] - b * sn[i];
+  };
   const int64_t slot = own_latent ? slots[t] : -1;
   const int R = kv_rank + rot_dim;
   if (slot >= 0) {
     T* crow = cache + static_cast<size_t>(slot) * R;
     for (int d = threadIdx.x; d < kv_rank; d += blockDim.x) st(crow + d, craw[d] * inv * latent_norm_w[d]);
-    for (int d = threadIdx.x; d < rot_dim; d += blockDim.x) {
-      float v = kraw[d];
-      if (d < rot_dims) {
-        const int i = d >> 1;
-        const float a = kraw[2 * i], b = kraw[2 * i + 1];
-        v = (d & 1) ? b * cs[i] + a * sn[i] : a * cs[i] - b * sn[i];
-      }
-      st(crow + kv_rank + d, v);
-    }
+    for (int d = threadIdx.x; d < rot_dim; d += blockDim.x) st(crow + kv_rank + d, turned(kraw, d));
   }
   const int hd = dim + rot_dim;
   for (int e = threadIdx.x; e < heads * hd; e += blockDim.x) {
@@ -81,14 +84,7 @@ __global__ void latent_prep_kernel(const float* __restrict__ qc, int ldq, T* __r
     if (d < dim) {
       st(q_plain + (static_cast<size_t>(t) * heads + h) * dim + d, qh[d]);
     } else {
-      const int r = d - dim;
-      float v = qh[d];
-      if (r < rot_dims) {
-        const int i = r >> 1;
-        const float a = qh[dim + 2 * i], b = qh[dim + 2 * i + 1];
-        v = (r & 1) ? b * cs[i] + a * sn[i] : a * cs[i] - b * sn[i];
-      }
-      q_full[(static_cast<size_t>(t) * heads + h) * R + kv_rank + r] = v;
+      q_full[(static_cast<size_t>(t) * heads + h) * R + kv_rank + d - dim] = turned(qh + dim, d - dim);
     }
   }
 }
@@ -207,20 +203,21 @@ __global__ void latent_attn_merge_kernel(T* __restrict__ out, const float* __res
   }
 }
 
-void launch_latent_prep(const float* qc, int ldq, void* q_plain, float* q_full, void* cache, const float* latent_norm_w,
-                        const double* rot_freq, float rot_mag, const int64_t* positions, const int64_t* slots, int T,
-                        int heads, int dim, int rot_dim, int rot_dims, int kv_rank, float eps, int dt, cudaStream_t st_) {
+void launch_latent_prep(const float* q, int ldq, const float* low, int ld_low, void* q_plain, float* q_full, void* cache,
+                        const float* latent_norm_w, const double* rot_freq, float rot_mag, int rot_half,
+                        const int64_t* positions, const int64_t* slots, int T, int heads, int dim, int rot_dim,
+                        int rot_dims, int kv_rank, float eps, int dt, cudaStream_t st_) {
   if (T <= 0) return;
   const size_t smem = (static_cast<size_t>(rot_dims) + 40) * 4;
   if (dt)
-    latent_prep_kernel<float><<<T, 256, smem, st_>>>(qc, ldq, (float*)q_plain, q_full, (float*)cache, latent_norm_w,
-                                                     rot_freq, rot_mag, positions, slots, heads, dim, rot_dim,
-                                                     rot_dims, kv_rank, eps);
+    latent_prep_kernel<float><<<T, 256, smem, st_>>>(q, ldq, low, ld_low, (float*)q_plain, q_full, (float*)cache,
+                                                     latent_norm_w, rot_freq, rot_mag, rot_half, positions, slots,
+                                                     heads, dim, rot_dim, rot_dims, kv_rank, eps);
   else
-    latent_prep_kernel<__nv_bfloat16><<<T, 256, smem, st_>>>(qc, ldq, (__nv_bfloat16*)q_plain, q_full,
+    latent_prep_kernel<__nv_bfloat16><<<T, 256, smem, st_>>>(q, ldq, low, ld_low, (__nv_bfloat16*)q_plain, q_full,
                                                              (__nv_bfloat16*)cache, latent_norm_w, rot_freq, rot_mag,
-                                                             positions, slots, heads, dim, rot_dim, rot_dims, kv_rank,
-                                                             eps);
+                                                             rot_half, positions, slots, heads, dim, rot_dim, rot_dims,
+                                                             kv_rank, eps);
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -577,8 +574,21 @@ void b200_latent_prep(const float* qc, int32_t ldq, void* q_plain, float* q_full
                      heads > 0 && dim >= 0 && rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim &&
                      rot_dims % 2 == 0 && kv_rank > 0 && (dt == 0 || dt == 1),
                  "latent_prep: bad arguments");
-  b200::launch_latent_prep(qc, ldq, q_plain, q_full, cache, latent_norm_w, rot_freq, rot_mag, positions, slot_mapping,
-                           num_tokens, heads, dim, rot_dim, rot_dims, kv_rank, eps, dt,
+  b200::launch_latent_prep(qc, ldq, qc + static_cast<size_t>(heads) * (dim + rot_dim), ldq, q_plain, q_full, cache,
+                           latent_norm_w, rot_freq, rot_mag, 0, positions, slot_mapping, num_tokens, heads, dim, rot_dim,
+                           rot_dims, kv_rank, eps, dt, reinterpret_cast<cudaStream_t>(stream));
+}
+void b200_latent_prep_ex(const float* q, int32_t ldq, const float* low, int32_t ld_low, void* q_plain, float* q_full,
+                         void* cache, const float* latent_norm_w, const double* rot_freq, float rot_mag,
+                         int32_t rot_half, const int64_t* positions, const int64_t* slot_mapping, int32_t num_tokens,
+                         int32_t heads, int32_t dim, int32_t rot_dim, int32_t rot_dims, int32_t kv_rank, float eps,
+                         int32_t dt, int64_t stream) {
+  B200_CHECK_ARG(q && q_plain && q_full && (!cache || (low && latent_norm_w && slot_mapping)) &&
+                     (rot_dims == 0 || rot_freq) && positions && heads > 0 && dim >= 0 && rot_dim >= 0 && rot_dims >= 0 &&
+                     rot_dims <= rot_dim && rot_dims % 2 == 0 && kv_rank > 0 && (dt == 0 || dt == 1),
+                 "latent_prep_ex: bad arguments");
+  b200::launch_latent_prep(q, ldq, low, ld_low, q_plain, q_full, cache, latent_norm_w, rot_freq, rot_mag, rot_half, positions,
+                           slot_mapping, num_tokens, heads, dim, rot_dim, rot_dims, kv_rank, eps, dt,
                            reinterpret_cast<cudaStream_t>(stream));
 }
 void b200_latent_prep_queries(const float* qc, int32_t ldq, void* q_plain, float* q_full, const double* rot_freq,
@@ -588,8 +598,9 @@ void b200_latent_prep_queries(const float* qc, int32_t ldq, void* q_plain, float
                      rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0 && kv_rank > 0 &&
                      (dt == 0 || dt == 1),
                  "latent_prep_queries: bad arguments");
-  b200::launch_latent_prep(qc, ldq, q_plain, q_full, nullptr, nullptr, rot_freq, rot_mag, positions, nullptr, num_tokens,
-                           heads, dim, rot_dim, rot_dims, kv_rank, 0.f, dt, reinterpret_cast<cudaStream_t>(stream));
+  b200::launch_latent_prep(qc, ldq, nullptr, 0, q_plain, q_full, nullptr, nullptr, rot_freq, rot_mag, 0, positions, nullptr,
+                           num_tokens, heads, dim, rot_dim, rot_dims, kv_rank, 0.f, dt,
+                           reinterpret_cast<cudaStream_t>(stream));
 }
 void b200_latent_attn_gated(void* out, const float* q_full, const void* cache, const float* sink, const float* gate,
                             int32_t ld_gate, const uint32_t* cu_seqlens_q, const uint32_t* context_lens,

@@ -7,12 +7,13 @@
 //              per-expert bias; with groups, the experts form equal runs of neighbours, a run's score is its largest
 //              choice score (or the sum of its two largest), and members of all but the `keep` best runs cannot be
 //              chosen.  Options: s = sigmoid(logit) per expert instead of the softmax; the chosen weights divided by
-//              their sum.
+//              their sum; or a choice by the largest (logit + bias), weighted by a softmax over the chosen ones only.
 //   sort     : pair p = token * top + choice; pairs are bucketed by expert into slots [off[e], off[e+1]).  The order
 //              inside a bucket is arbitrary and does not influence any result: every pair is one independent row.
 //   gate_up  : act[slot, f] = silu(h[token] . Wg[e, f]) * (h[token] . Wu[e, f]);  W_gate_up [E, 2F, width] (gate rows
 //              first), h in the activation dtype, fp32 accumulation, act stored in the activation dtype.  Ungated
-//              experts: act[slot, f] = relu(h[token] . Wu[e, f])^2, W_up [E, F, width].
+//              experts: act[slot, f] = relu(h[token] . Wu[e, f])^2, W_up [E, F, width].  Clamped gated experts:
+//              g = min(h . Wg, limit), u = clamp(h . Wu, -limit, limit), act = g sigmoid(alpha g) (u + up_add).
 //   down     : y[slot, d] = act[slot] . Wd[e, d];  W_down [E, width, F]; fp32 out.
 //   combine  : x[token] (+)= sum_choice w[token, choice] * y[slot(token, choice)], choices added in order (no atomics).
 //              Router outputs past the last real expert are identity experts: y = the token's own input row.
@@ -53,12 +54,14 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
       s[e] = p;
       c[e] = p + (bias ? bias[e] : 0.f);
     }
-  } else {
+  } else if (score == 1) {
     for (int e = lane; e < E; e += 32) {
       const float p = sigmoid_f(z[e]);
       s[e] = p;
       c[e] = p + (bias ? bias[e] : 0.f);
     }
+  } else {                         // the logits themselves; they become weights once the choice is known
+    for (int e = lane; e < E; e += 32) s[e] = c[e] = z[e] + (bias ? bias[e] : 0.f);
   }
   __syncwarp();
   if (groups > 0) {
@@ -82,6 +85,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
     __syncwarp();
   }
   float total = 0.f;             // sum of the chosen scores
+  float top_z = 0.f;             // (score 2) the first chosen logit, the largest of all that are chosen
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
     int bi = E;
@@ -102,16 +106,18 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
       }
     }
     if (bi >= E) bi = 0;       // fewer available experts than `top` (rejected by the launcher; keeps the index valid)
-    total += s[bi];
+    if (j == 0) top_z = s[bi];
+    const float wt = score == 2 ? expf(s[bi] - top_z) : s[bi];
+    total += wt;
     if (lane == 0) {
       top_idx[static_cast<size_t>(t) * top + j] = bi;
-      top_w[static_cast<size_t>(t) * top + j] = s[bi] * scale;
+      top_w[static_cast<size_t>(t) * top + j] = wt * scale;
       c[bi] = -INFINITY;
     }
     __syncwarp();
   }
-  if (renorm)
-    for (int j = lane; j < top; j += 32) top_w[static_cast<size_t>(t) * top + j] /= total + 1e-20f;
+  if (renorm || score == 2)
+    for (int j = lane; j < top; j += 32) top_w[static_cast<size_t>(t) * top + j] /= total + (score == 2 ? 0.f : 1e-20f);
 }
 
 // single block: histogram, exclusive scan, scatter
@@ -162,14 +168,22 @@ __device__ __forceinline__ bool find_tile(const int32_t* __restrict__ off, int E
 }
 
 // ACT: 0 = plain product over slot rows, fp32 out (the down projection); 1 = gathered token rows, two weight matrices,
-// SiLU(gate) * up; 2 = gathered token rows, one matrix, relu(.)^2.  ACT != 0 stores the activation dtype.
+// SiLU(gate) * up; 2 = gathered token rows, one matrix, relu(.)^2; 3 = as 1 with the clamped gate.  ACT != 0 stores the
+// activation dtype.
+template <int ACT>
+__device__ __forceinline__ float expert_gate(float g, float u, const b200_expert_act& p) {
+  if (ACT != 3) return silu_exact(g) * u;
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit);
+  return g / (1.f + expf(-p.alpha * g)) * (u + p.up_add);
+}
 // fp32 path (and the generic one): 256 threads, each 2 rows x 2 columns (x 2 matrices when gated)
 template <typename T, int ACT>
 __global__ void __launch_bounds__(256)
 grouped_linear_fma_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __restrict__ w,
                           const int32_t* __restrict__ off, const int32_t* __restrict__ pair_of_slot, int top, int E,
-                          int K, int N) {
-  constexpr bool GATED = ACT == 1, GATHER = ACT != 0;
+                          int K, int N, const b200_expert_act actp) {
+  constexpr bool GATED = ACT == 1 || ACT == 3, GATHER = ACT != 0;
   __shared__ float As[TM][TK + 1], W0[TN][TK + 1], W1[GATED ? TN : 1][TK + 1];
   int e, s0, rows;
   if (!find_tile(off, E, blockIdx.x, &e, &s0, &rows)) return;
@@ -215,7 +229,7 @@ grouped_linear_fma_kernel(void* __restrict__ out_, const T* __restrict__ a, cons
       if (r < rows && n < N) {
         const size_t o = static_cast<size_t>(s0 + r) * N + n;
         if (GATED) {
-          st(reinterpret_cast<T*>(out_) + o, silu_exact(acc0[i][j]) * acc1[i][j]);
+          st(reinterpret_cast<T*>(out_) + o, expert_gate<ACT>(acc0[i][j], acc1[i][j], actp));
         } else if (ACT == 2) {
           const float u = fmaxf(acc0[i][j], 0.f);
           st(reinterpret_cast<T*>(out_) + o, u * u);
@@ -248,8 +262,9 @@ template <int ACT>
 __global__ void __launch_bounds__(128)
 grouped_linear_mma_kernel(void* __restrict__ out_, const __nv_bfloat16* __restrict__ a,
                           const __nv_bfloat16* __restrict__ w, const int32_t* __restrict__ off,
-                          const int32_t* __restrict__ pair_of_slot, int top, int E, int K, int N) {
-  constexpr bool GATED = ACT == 1, GATHER = ACT != 0;
+                          const int32_t* __restrict__ pair_of_slot, int top, int E, int K, int N,
+                          const b200_expert_act actp) {
+  constexpr bool GATED = ACT == 1 || ACT == 3, GATHER = ACT != 0;
   // two stages: the 16-byte asynchronous copies of K chunk i + 1 run under the MMAs of chunk i
   __shared__ __align__(16) __nv_bfloat16 As[2][TM][MP], W0[2][MN][MP], W1[2][GATED ? MN : 1][MP];
   __shared__ size_t arow[TM];
@@ -348,7 +363,7 @@ grouped_linear_mma_kernel(void* __restrict__ out_, const __nv_bfloat16* __restri
           const size_t o = static_cast<size_t>(s0 + r) * N + n;
           if (GATED) {
             reinterpret_cast<__nv_bfloat16*>(out_)[o] =
-                __float2bfloat16_rn(silu_exact(acc0[hf][nb][f]) * acc1[hf][nb][f]);
+                __float2bfloat16_rn(expert_gate<ACT>(acc0[hf][nb][f], acc1[hf][nb][f], actp));
           } else if (ACT == 2) {
             const float u = fmaxf(acc0[hf][nb][f], 0.f);
             reinterpret_cast<__nv_bfloat16*>(out_)[o] = __float2bfloat16_rn(u * u);
@@ -383,7 +398,7 @@ void launch_moe_route(const float* logits, const float* bias, int T, int E, int 
                       int group_top, int renorm, float scale, int32_t* top_idx, float* top_w, cudaStream_t st_) {
   if (T <= 0) return;
   if (group_top == 0) group_top = 1;
-  if (score < 0 || score > 1 || group_top < 1 || group_top > 2) {
+  if (score < 0 || score > 2 || group_top < 1 || group_top > 2) {
     set_error(1, "moe_route: unknown score, or a group score of more than two members");
     return;
   }
@@ -427,27 +442,30 @@ static bool use_mma() {
 
 template <int ACT>
 static void grouped_linear(void* out, const void* a, const void* w, const int32_t* off, const int32_t* pair_of_slot,
-                           int pairs, int top, int E, int K, int N, int dt, cudaStream_t st_) {
+                           int pairs, int top, int E, int K, int N, int dt, cudaStream_t st_,
+                           const b200_expert_act& act = b200_expert_act{}) {
   if (pairs <= 0) return;
   const int tiles = (pairs + TM - 1) / TM + E;
   if (dt) {
     grouped_linear_fma_kernel<float, ACT><<<dim3(tiles, (N + TN - 1) / TN), 256, 0, st_>>>(
-        out, (const float*)a, (const float*)w, off, pair_of_slot, top, E, K, N);
+        out, (const float*)a, (const float*)w, off, pair_of_slot, top, E, K, N, act);
   } else if (use_mma()) {
     grouped_linear_mma_kernel<ACT><<<dim3(tiles, (N + MN - 1) / MN), 128, 0, st_>>>(
-        out, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, off, pair_of_slot, top, E, K, N);
+        out, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, off, pair_of_slot, top, E, K, N, act);
   } else {
     grouped_linear_fma_kernel<__nv_bfloat16, ACT><<<dim3(tiles, (N + TN - 1) / TN), 256, 0, st_>>>(
-        out, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, off, pair_of_slot, top, E, K, N);
+        out, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, off, pair_of_slot, top, E, K, N, act);
   }
   B200_CUDA_LAUNCH_CHECK();
 }
 
 void launch_moe_gate_up(void* act_out, const void* h, const void* w_up, const int32_t* expert_off,
-                        const int32_t* pair_of_slot, int pairs, int top, int E, int width, int ff, int act, int dt,
-                        cudaStream_t st_) {
-  if (act == 0)
+                        const int32_t* pair_of_slot, int pairs, int top, int E, int width, int ff,
+                        const b200_expert_act& act, int dt, cudaStream_t st_) {
+  if (act.kind == B200_EXPERT_SILU)
     grouped_linear<1>(act_out, h, w_up, expert_off, pair_of_slot, pairs, top, E, width, ff, dt, st_);
+  else if (act.kind == B200_EXPERT_CLAMPED)
+    grouped_linear<3>(act_out, h, w_up, expert_off, pair_of_slot, pairs, top, E, width, ff, dt, st_, act);
   else
     grouped_linear<2>(act_out, h, w_up, expert_off, pair_of_slot, pairs, top, E, width, ff, dt, st_);
 }
@@ -502,7 +520,7 @@ int64_t b200_moe_workspace_bytes(int32_t num_tokens, int32_t experts, int32_t to
 namespace b200 {
 // buckets, both grouped products; the rows of the (token, choice) pairs and their places stay in the workspace
 static void moe_expert_rows(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down, int T, int experts,
-                            int identity, int top, int width, int ff, int act, int dt, void* workspace,
+                            int identity, int top, int width, int ff, const b200_expert_act& act, int dt, void* workspace,
                             const float** down_out, const int32_t** slot_out, cudaStream_t st_) {
   const int P = T * top, all = experts + identity;
   auto up = [](size_t v) { return (v + 255) / 256 * 256; };
@@ -522,30 +540,51 @@ static void moe_expert_rows(const void* h, const int32_t* top_idx, const void* w
 }  // namespace b200
 
 extern "C" {
-void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, const float* top_w, const void* w_up,
-                         const void* w_down, int32_t num_tokens, int32_t experts, int32_t identity, int32_t top,
-                         int32_t width, int32_t ff, int32_t act, int32_t accumulate, const void* ident,
-                         int32_t ident_f32, int32_t dt, void* workspace, int64_t stream) {
+static bool expert_act_ok(const b200_expert_act* a) {
+  return a && a->kind >= B200_EXPERT_SILU && a->kind <= B200_EXPERT_CLAMPED && (a->kind != B200_EXPERT_CLAMPED || a->limit >= 0.f);
+}
+void b200_moe_experts_act(float* out, const void* h, const int32_t* top_idx, const float* top_w, const void* w_up,
+                          const void* w_down, int32_t num_tokens, int32_t experts, int32_t identity, int32_t top,
+                          int32_t width, int32_t ff, const b200_expert_act* act, int32_t accumulate, const void* ident,
+                          int32_t ident_f32, int32_t dt, void* workspace, int64_t stream) {
   B200_CHECK_ARG(out && h && top_idx && top_w && w_up && w_down && workspace && (dt == 0 || dt == 1) &&
-                     (act == 0 || act == 1) && identity >= 0 && (identity == 0 || ident),
+                     expert_act_ok(act) && identity >= 0 && (identity == 0 || ident),
                  "moe_experts: bad arguments");
   cudaStream_t st_ = reinterpret_cast<cudaStream_t>(stream);
   const float* down = nullptr;
   const int32_t* sop = nullptr;
-  b200::moe_expert_rows(h, top_idx, w_up, w_down, num_tokens, experts, identity, top, width, ff, act, dt, workspace, &down,
+  b200::moe_expert_rows(h, top_idx, w_up, w_down, num_tokens, experts, identity, top, width, ff, *act, dt, workspace, &down,
                         &sop, st_);
   b200::launch_moe_combine(out, down, sop, top_idx, top_w, num_tokens, top, width, experts, identity ? ident : nullptr,
                            ident_f32, dt, accumulate, st_);
+}
+void b200_moe_experts_ex(float* out, const void* h, const int32_t* top_idx, const float* top_w, const void* w_up,
+                         const void* w_down, int32_t num_tokens, int32_t experts, int32_t identity, int32_t top,
+                         int32_t width, int32_t ff, int32_t act, int32_t accumulate, const void* ident,
+                         int32_t ident_f32, int32_t dt, void* workspace, int64_t stream) {
+  B200_CHECK_ARG(act == B200_EXPERT_SILU || act == B200_EXPERT_RELU2, "moe_experts: this call takes kinds without constants");
+  const b200_expert_act a{act, 0.f, 0.f, 0.f};
+  b200_moe_experts_act(out, h, top_idx, top_w, w_up, w_down, num_tokens, experts, identity, top, width, ff, &a, accumulate,
+                       ident, ident_f32, dt, workspace, stream);
+}
+void b200_moe_experts_rows_act(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down,
+                               int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff,
+                               const b200_expert_act* act, int32_t dt, void* workspace, const float** down,
+                               const int32_t** slot_of_pair, int64_t stream) {
+  B200_CHECK_ARG(h && top_idx && w_up && w_down && workspace && down && slot_of_pair && (dt == 0 || dt == 1) &&
+                     expert_act_ok(act),
+                 "moe_experts_rows: bad arguments");
+  b200::moe_expert_rows(h, top_idx, w_up, w_down, num_tokens, experts, 0, top, width, ff, *act, dt, workspace, down,
+                        slot_of_pair, reinterpret_cast<cudaStream_t>(stream));
 }
 void b200_moe_experts_rows(const void* h, const int32_t* top_idx, const void* w_up, const void* w_down,
                            int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff, int32_t act,
                            int32_t dt, void* workspace, const float** down, const int32_t** slot_of_pair,
                            int64_t stream) {
-  B200_CHECK_ARG(h && top_idx && w_up && w_down && workspace && down && slot_of_pair && (dt == 0 || dt == 1) &&
-                     (act == 0 || act == 1),
-                 "moe_experts_rows: bad arguments");
-  b200::moe_expert_rows(h, top_idx, w_up, w_down, num_tokens, experts, 0, top, width, ff, act, dt, workspace, down,
-                        slot_of_pair, reinterpret_cast<cudaStream_t>(stream));
+  B200_CHECK_ARG(act == B200_EXPERT_SILU || act == B200_EXPERT_RELU2, "moe_experts_rows: this call takes kinds without constants");
+  const b200_expert_act a{act, 0.f, 0.f, 0.f};
+  b200_moe_experts_rows_act(h, top_idx, w_up, w_down, num_tokens, experts, top, width, ff, &a, dt, workspace, down,
+                            slot_of_pair, stream);
 }
 void b200_moe_experts(float* x, const void* h, const int32_t* top_idx, const float* top_w, const void* w_gate_up,
                       const void* w_down, int32_t num_tokens, int32_t experts, int32_t top, int32_t width, int32_t ff,

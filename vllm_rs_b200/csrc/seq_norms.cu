@@ -1,7 +1,8 @@
 // Row kernels of decoders that keep the residual stream in fp32: embedding lookup into the stream, RMS norm of the
 // stream (weight stored either plainly or as an offset from one), the grouped RMS norm with a SiLU gate that follows
 // a recurrent mixer (gate applied before or after the normalisation), SiLU * mul over an fp32 gate|up block, and
-// the rounding of fp32 rows to the dtype that feeds the next matrix product, the norm of the stream with a choice of
+// the rounding of fp32 rows to the dtype that feeds the next matrix product (with or without a sigmoid gate per element),
+// rotary positions on rows that stay in fp32, the norm of the stream with a choice of
 // kind (RMS / dynamic tanh / layer norm) and a token shift, the weighted sum of the stored results of earlier layers, and
 // the step between two sublayers of hyper-connected streams (update, read, norm).  All arithmetic is fp32; the output
 // dtype is bf16 or fp32.  Beside the fp16 / bf16 row kernels of glue.cu (rmsnorm_kernel, silu_mul_kernel), which
@@ -38,13 +39,14 @@ __global__ void embed_f32_kernel(float* __restrict__ x, const T* __restrict__ ta
   }
 }
 
-// out[r] = x[row(r)] / sqrt(mean(x^2) + eps) * (w_offset + w); rows == nullptr: row(r) = r
+// out[r] = x[row(r)] / sqrt(mean(x^2) + eps) * (w_offset + w); rows == nullptr: row(r) = r; ldx: row stride of x
 template <typename T>
-__global__ void resid_rmsnorm_kernel(T* __restrict__ out, const float* __restrict__ x, const float* __restrict__ w,
-                                     int width, float eps, float w_offset, const uint32_t* __restrict__ rows) {
+__global__ void resid_rmsnorm_kernel(T* __restrict__ out, const float* __restrict__ x, size_t ldx,
+                                     const float* __restrict__ w, int width, float eps, float w_offset,
+                                     const uint32_t* __restrict__ rows) {
   __shared__ float red[33];
   const int r = blockIdx.x;
-  const float* xr = x + static_cast<size_t>(rows ? rows[r] : r) * width;
+  const float* xr = x + static_cast<size_t>(rows ? rows[r] : r) * ldx;
   float ss = 0.f;
   for (int d = threadIdx.x; d < width; d += blockDim.x) ss += xr[d] * xr[d];
   ss = block_sum(ss, red);
@@ -124,6 +126,35 @@ __global__ void silu_mul_f32_kernel(T* __restrict__ out, const float* __restrict
   }
 }
 
+// Rotary positions on `heads` neighbouring heads of an fp32 row, in place (the queries and keys of a recurrent mixer, which
+// go into the scan as they lie in the projection row).  One block per token: cos / sin of the token's angles (angles in
+// double) are made once in shared memory and serve every head.  Pairs are (i, i + rot_dims / 2) or interleaved (2i, 2i+1).
+__global__ void rotary_rows_kernel(float* __restrict__ x, int ld, const double* __restrict__ rot_freq, float rot_mag,
+                                   int rot_half, const int64_t* __restrict__ positions, int heads, int dim,
+                                   int rot_dims) {
+  extern __shared__ float sm[];          // cos[rot_dims / 2] | sin[rot_dims / 2]
+  const int t = blockIdx.x, half = rot_dims / 2;
+  float* cs = sm;
+  float* sn = sm + half;
+  const double pos = static_cast<double>(positions[t]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    double s, c;
+    sincos(pos * rot_freq[i], &s, &c);
+    cs[i] = static_cast<float>(c) * rot_mag;
+    sn[i] = static_cast<float>(s) * rot_mag;
+  }
+  __syncthreads();
+  float* row = x + static_cast<size_t>(t) * ld;
+  for (int e = threadIdx.x; e < heads * half; e += blockDim.x) {
+    const int h = e / half, i = e - h * half;
+    float* a = row + static_cast<size_t>(h) * dim + (rot_half ? i : 2 * i);
+    float* b = a + (rot_half ? half : 1);
+    const float u = *a, v = *b;
+    *a = u * cs[i] - v * sn[i];
+    *b = v * cs[i] + u * sn[i];
+  }
+}
+
 // V consecutive fp32 values of a thread (16-byte accesses for V = 4), stored as fp32 or rounded to bf16
 template <int V> struct FloatVec;
 template <> struct FloatVec<1> {
@@ -146,6 +177,22 @@ template <int V> __device__ __forceinline__ void store_vec(__nv_bfloat16* p, con
     *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(q);
   } else {
     *p = __float2bfloat16_rn(f.v[0]);
+  }
+}
+
+// out[t, d] = in[t, d] * sigmoid(gate[t, d]) in the operand dtype; grid.x covers the columns (V per thread), grid.y the rows
+template <typename T, int V>
+__global__ void gate_rows_kernel(T* __restrict__ out, const float* __restrict__ in, const float* __restrict__ gate,
+                                 int ld_gate, int n, int rows) {
+  const int d = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (d >= n) return;
+  for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+    FloatVec<V> z, g;
+    z.load(in + static_cast<size_t>(t) * n + d);
+    g.load(gate + static_cast<size_t>(t) * ld_gate + d);
+#pragma unroll
+    for (int c = 0; c < V; ++c) z.v[c] *= sigmoid_f(g.v[c]);
+    store_vec<V>(out + static_cast<size_t>(t) * n + d, z);
   }
 }
 
@@ -264,9 +311,9 @@ __global__ void hyper_step_kernel(const HyperArgs a) {
   float* u = sm + ((36 + S * S + 2 * S + 2 * a.top + 3) & ~3);
   const size_t t = a.rows ? a.rows[r] : r;
   const bool update = a.y != nullptr || a.down != nullptr;
-  for (int i = threadIdx.x; i < S * S; i += blockDim.x) mix[i] = update ? a.mix[i] : 0.f;
+  for (int i = threadIdx.x; i < S * S; i += blockDim.x) mix[i] = update ? (a.mix ? a.mix[i] : (i % (S + 1) == 0 ? 1.f : 0.f)) : 0.f;
   for (int i = threadIdx.x; i < S; i += blockDim.x) {
-    ow[i] = update ? a.out_w[i] : 0.f;
+    ow[i] = update ? (a.out_w ? a.out_w[i] : 1.f) : 0.f;
     iw[i] = a.in_w ? a.in_w[i] : 1.f;
   }
   for (int i = threadIdx.x; i < a.top; i += blockDim.x) {
@@ -393,12 +440,13 @@ void launch_embed_f32(float* x, const void* table, const uint32_t* ids, const in
 }
 
 void launch_resid_rmsnorm(void* out, const float* x, const float* w, int T, int width, float eps, float w_offset,
-                          const uint32_t* rows, int dt, cudaStream_t st_) {
+                          const uint32_t* rows, int dt, cudaStream_t st_, int ldx) {
   if (T <= 0) return;
+  if (ldx == 0) ldx = width;
   if (dt)
-    resid_rmsnorm_kernel<float><<<T, 256, 0, st_>>>((float*)out, x, w, width, eps, w_offset, rows);
+    resid_rmsnorm_kernel<float><<<T, 256, 0, st_>>>((float*)out, x, ldx, w, width, eps, w_offset, rows);
   else
-    resid_rmsnorm_kernel<__nv_bfloat16><<<T, 256, 0, st_>>>((__nv_bfloat16*)out, x, w, width, eps, w_offset, rows);
+    resid_rmsnorm_kernel<__nv_bfloat16><<<T, 256, 0, st_>>>((__nv_bfloat16*)out, x, ldx, w, width, eps, w_offset, rows);
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -468,6 +516,28 @@ void launch_ff_act(void* out, const float* up, int ld, int T, int ff, int gate_c
   else go((TYPE*)out, act == 1 ? ff_act_kernel<TYPE, 1, 1> : ff_act_kernel<TYPE, 2, 1>);
   if (dt) { B200_FF_ACT(float) } else { B200_FF_ACT(__nv_bfloat16) }
 #undef B200_FF_ACT
+  B200_CUDA_LAUNCH_CHECK();
+}
+
+void launch_rotary_rows(float* x, int ld, const double* rot_freq, float rot_mag, int rot_half, const int64_t* positions,
+                        int T, int heads, int dim, int rot_dims, cudaStream_t st_) {
+  if (T <= 0 || heads <= 0 || rot_dims <= 0) return;
+  const int pairs = heads * (rot_dims / 2);
+  const int threads = pairs >= 1024 ? 512 : (pairs >= 256 ? 256 : 128);
+  rotary_rows_kernel<<<T, threads, static_cast<size_t>(rot_dims) * 4, st_>>>(x, ld, rot_freq, rot_mag, rot_half, positions,
+                                                                             heads, dim, rot_dims);
+  B200_CUDA_LAUNCH_CHECK();
+}
+
+void launch_gate_rows(void* out, const float* in, const float* gate, int ld_gate, int T, int n, int dt, cudaStream_t st_) {
+  if (T <= 0 || n <= 0) return;
+  const bool vec = n % 4 == 0 && ld_gate % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(gate)) % 16 == 0;
+  const int per_block = 256 * (vec ? 4 : 1);
+  const dim3 grid((n + per_block - 1) / per_block, std::min(T, 32768));
+  auto go = [&](auto* o, auto kern) { kern<<<grid, 256, 0, st_>>>(o, in, gate, ld_gate, n, T); };
+  if (dt) go((float*)out, vec ? gate_rows_kernel<float, 4> : gate_rows_kernel<float, 1>);
+  else go((__nv_bfloat16*)out, vec ? gate_rows_kernel<__nv_bfloat16, 4> : gate_rows_kernel<__nv_bfloat16, 1>);
   B200_CUDA_LAUNCH_CHECK();
 }
 
@@ -567,6 +637,25 @@ void b200_resid_add_rmsnorm(float* x, const float* y, const float* w, int32_t nu
   b200::launch_resid_add_rmsnorm(x, y, w, num_tokens, width, eps, w_offset, nullptr,
                                  reinterpret_cast<cudaStream_t>(stream));
 }
+void b200_rmsnorm_rows(void* out, const float* x, int32_t ldx, const float* w, int32_t num_tokens, int32_t n, float eps,
+                       float w_offset, int32_t dt, int64_t stream) {
+  B200_CHECK_ARG(out && x && w && n > 0 && ldx >= n && (dt == 0 || dt == 1), "rmsnorm_rows: bad arguments");
+  b200::launch_resid_rmsnorm(out, x, w, num_tokens, n, eps, w_offset, nullptr, dt, reinterpret_cast<cudaStream_t>(stream), ldx);
+}
+void b200_rotary_rows(float* x, int32_t ld, const double* rot_freq, float rot_mag, int32_t rot_half,
+                      const int64_t* positions, int32_t num_tokens, int32_t heads, int32_t dim, int32_t rot_dims,
+                      int64_t stream) {
+  B200_CHECK_ARG(x && positions && heads > 0 && dim > 0 && ld >= heads * dim && rot_dims >= 0 && rot_dims <= dim &&
+                     rot_dims % 2 == 0 && (rot_dims == 0 || rot_freq),
+                 "rotary_rows: bad arguments");
+  b200::launch_rotary_rows(x, ld, rot_freq, rot_mag, rot_half, positions, num_tokens, heads, dim, rot_dims,
+                           reinterpret_cast<cudaStream_t>(stream));
+}
+void b200_gate_rows(void* out, const float* in, const float* gate, int32_t ld_gate, int32_t num_tokens, int32_t n,
+                    int32_t dt, int64_t stream) {
+  B200_CHECK_ARG(out && in && gate && n > 0 && ld_gate >= n && (dt == 0 || dt == 1), "gate_rows: bad arguments");
+  b200::launch_gate_rows(out, in, gate, ld_gate, num_tokens, n, dt, reinterpret_cast<cudaStream_t>(stream));
+}
 void b200_stream_norm(void* out, const float* x, const float* w, const float* bias, float alpha, int32_t kind,
                       float eps, float w_offset, const uint32_t* rows, const float* shift_w, float* shift_state,
                       const int32_t* state_slots, const uint32_t* cu_seqlens_q, const uint32_t* context_lens,
@@ -584,7 +673,7 @@ void b200_hyper_step(void* out, float* x_out, int64_t out_stride, const float* x
                      float eps, float w_offset, const uint32_t* rows, int32_t streams, int32_t num_tokens, int32_t width,
                      int32_t dt, int64_t stream) {
   B200_CHECK_ARG((out || x_out) && x_in && width > 0 && (dt == 0 || dt == 1) && in_stride >= 0 && out_stride >= 0 &&
-                     (!out || w) && (!(y || down) || (mix && out_w)) && (!down || (slot_of_pair && top_w && top > 0)) &&
+                     (!out || w) && (!down || (slot_of_pair && top_w && top > 0)) &&
                      (!rows || !x_out) && kind >= B200_NORM_RMS && kind <= B200_NORM_LAYER,
                  "hyper_step: bad arguments");
   b200::launch_hyper_step(out, x_out, static_cast<size_t>(out_stride), x_in, static_cast<size_t>(in_stride), y, down,

@@ -75,7 +75,7 @@ __device__ __forceinline__ int seq_of_row(const uint32_t* __restrict__ cu, int n
 void launch_embed_f32(float* x, const void* table, const uint32_t* ids, const int64_t* positions, float pos_base, int T,
                       int width, int vocab, float scale, int dt, void* cast_out, cudaStream_t st);
 void launch_resid_rmsnorm(void* out, const float* x, const float* w, int T, int width, float eps, float w_offset,
-                          const uint32_t* rows, int dt, cudaStream_t st);
+                          const uint32_t* rows, int dt, cudaStream_t st, int ldx = 0);      // ldx 0: width
 void launch_gated_group_norm(void* out, const float* y, int ldy, const float* gate, int ldg, const float* w, int w_period,
                              int T, int C, int group, float eps, int gate_first, int gate_act, int dt, cudaStream_t st);
 // cast_out (may be NULL): the updated rows rounded to bf16 as well
@@ -83,6 +83,11 @@ void launch_resid_add_rmsnorm(float* x, const float* y, const float* w, int T, i
                               void* cast_out, cudaStream_t st);
 void launch_bias_rows(float* y, const float* bias, float scale, int T, int n, cudaStream_t st);
 void launch_cast_rows(void* out, const float* in, int ld_in, int T, int n, int dt, cudaStream_t st);
+// out [T, n] = in * sigmoid(gate), in fp32 [T, n], gate fp32 with row stride ld_gate
+void launch_gate_rows(void* out, const float* in, const float* gate, int ld_gate, int T, int n, int dt, cudaStream_t st);
+// rotary positions on `heads` heads of `dim` entries in place (fp32 rows with stride ld)
+void launch_rotary_rows(float* x, int ld, const double* rot_freq, float rot_mag, int rot_half, const int64_t* positions,
+                        int T, int heads, int dim, int rot_dims, cudaStream_t st);
 void launch_silu_mul_f32(void* out, const float* gate_up, int T, int ff, int dt, cudaStream_t st);
 // out [T, ff] = act(up[t, d] + bias[d]) (* sigmoid(up[t, gate_col]) when gate_col >= 0); act 1: relu(.)^2, 2: exact GELU;
 // up fp32 with row stride ld; bias (may be NULL): fp32 [ff]
@@ -101,10 +106,13 @@ void launch_hyper_step(void* out, float* x_out, size_t out_stride, const float* 
                        float eps, float w_offset, const uint32_t* rows, int streams, int T, int width, int dt,
                        cudaStream_t st);
 
-void launch_latent_prep(const float* qc, int ldq, void* q_plain, float* q_full, void* cache, const float* latent_norm_w,
-                        const double* rot_freq, float rot_mag, const int64_t* positions, const int64_t* slots, int T,
-                        int heads, int dim, int rot_dim, int rot_dims, int kv_rank, float eps, int dt, cudaStream_t st);
-// cache == nullptr: the row holds queries only (a layer that reads another layer's cache); gate: per-head output gate
+// q [T, ldq]: the queries; low [T, ld_low]: raw latent | raw rotated key part (often the same rows, behind the queries).
+// cache == nullptr: queries only (a layer that reads another layer's cache)
+void launch_latent_prep(const float* q, int ldq, const float* low, int ld_low, void* q_plain, float* q_full, void* cache,
+                        const float* latent_norm_w, const double* rot_freq, float rot_mag, int rot_half,
+                        const int64_t* positions, const int64_t* slots, int T, int heads, int dim, int rot_dim,
+                        int rot_dims, int kv_rank, float eps, int dt, cudaStream_t st);
+// gate: per-head output gate
 void launch_latent_attn(void* out, const float* q_full, const void* cache, const float* sink, const float* gate,
                         int ld_gate, const uint32_t* cu, const uint32_t* ctx, const uint32_t* block_tables,
                         int max_blocks, int num_seqs, int T, int heads, int kv_rank, int rot_dim, int window, float scale,
@@ -149,15 +157,16 @@ void launch_decay_attn(float* out, const float* q, const float* k, const float* 
                        const int32_t* slots, const uint32_t* cu, const uint32_t* ctx, int num_seqs, int heads, int dim,
                        int vdim, cudaStream_t st);
 
-// score 0 softmax, 1 sigmoid; group_top: a group's score sums its 1 or 2 best members; renorm: weights / (their sum + 1e-20)
+// score 0 softmax, 1 sigmoid, 2 logits + bias with a softmax over the chosen ones; group_top: a group's score sums its 1 or
+// 2 best members; renorm: weights / (their sum + 1e-20)
 void launch_moe_route(const float* logits, const float* bias, int T, int E, int top, int groups, int keep, int score,
                       int group_top, int renorm, float scale, int32_t* top_idx, float* top_w, cudaStream_t st);
 void launch_moe_sort(const int32_t* top_idx, int pairs, int E, int32_t* expert_off, int32_t* pair_of_slot,
                      int32_t* slot_of_pair, cudaStream_t st);
-// act 0: SiLU(gate) * up over [gate | up] rows; act 1: relu(up)^2 over up rows
+// act.kind: B200_EXPERT_*
 void launch_moe_gate_up(void* act_out, const void* h, const void* w_up, const int32_t* expert_off,
-                        const int32_t* pair_of_slot, int pairs, int top, int E, int width, int ff, int act, int dt,
-                        cudaStream_t st);
+                        const int32_t* pair_of_slot, int pairs, int top, int E, int width, int ff,
+                        const b200_expert_act& act, int dt, cudaStream_t st);
 void launch_moe_down(float* out, const void* act, const void* w_down, const int32_t* expert_off, int pairs, int E,
                      int width, int ff, int dt, cudaStream_t st);
 // x = (accumulate ? x : 0) + sum of the choices; choices >= E are identity experts and read `ident`

@@ -24,6 +24,7 @@ from ._lib import HybridConfig, HybridLayer
 MIXER_LATENT_ATTN, MIXER_DELTA_RULE, MIXER_SSD, MIXER_WINDOW_ATTN, MIXER_DECAY_ATTN = 0, 1, 2, 3, 4
 LAYOUT_PARALLEL, LAYOUT_SANDWICH, LAYOUT_POSTNORM, LAYOUT_PRENORM, LAYOUT_HYPER = 0, 1, 2, 3, 4
 NORM_RMS, NORM_DYNTANH, NORM_LAYER = 0, 1, 2
+EXPERT_SILU, EXPERT_RELU2, EXPERT_CLAMPED = 0, 1, 2
 MAX_STREAMS = 16
 PAGE = 64
 
