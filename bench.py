@@ -38,6 +38,12 @@ Configs (BASELINE.json `configs`):
                       routers; fp32 streams, bf16 operands, random weights) next to the Gibevik decoder of equal width,
                       depth and expert sizes: prefill and decode tokens/s of both, and each kernel alone beside the like
                       kernel of the other models (vllm_rs_b200/bench_zufulix.py).
+  sonalix             the Sonalix decoder (pre-norm layers with dynamic-tanh norms; windowed attention with a learned sink,
+                      capped scores and mixed values; retention; latent attention with latent queries and an element
+                      gate; dense and routed clamped feed-forwards; fp32 residual, bf16 operands, random weights) next to
+                      the Gibevik and Fidasun decoders of equal width, depth and expert sizes: prefill and decode
+                      tokens/s of all, and each kernel alone beside the like kernel of the other models
+                      (vllm_rs_b200/bench_sonalix.py).
 
 Keys of the JSON line:
   value  device-resident: step inputs already in HBM, K CUDA-graph replays of the SAME step (the same KV slot is
@@ -79,6 +85,7 @@ CONFIGS = {
     "gibevik": dict(model="gibevik", fmt="bf16", kind="hybrid", baseline=None, label="Gibevik decoder"),
     "tasadra": dict(model="tasadra", fmt="bf16", kind="hybrid", baseline=None, label="Tasadra decoder"),
     "zufulix": dict(model="zufulix", fmt="bf16", kind="hybrid", baseline=None, label="Zufulix decoder"),
+    "sonalix": dict(model="sonalix", fmt="bf16", kind="hybrid", baseline=None, label="Sonalix decoder"),
     "l70_tp8": dict(model="llama3-70b", fmt="awq", kind="serve", gpus=8, max_num_seqs=64, requests=96,
                     prompt=(512, 2048), max_tokens=64, mean_gap_steps=1.0, baseline="configs[4]",
                     label="Llama-3-70B AWQ-int4"),
@@ -102,7 +109,7 @@ def parse():
     ap.add_argument("--no-extra-configs", action="store_true", help="N = 4 / 8: skip the q72_tp4 / l70_tp8 legs")
     ap.add_argument("--py-step", action="store_true",
                     help="e2e: drive the step from Python over the individual C symbols instead of b200_engine_step")
-    ap.add_argument("--size", default="w2048,w4096", help="--config fidasun / zalalix / gibevik / tasadra / zufulix: layer sizes, comma separated")
+    ap.add_argument("--size", default="w2048,w4096", help="--config fidasun / zalalix / gibevik / tasadra / zufulix / sonalix: layer sizes, comma separated")
     ap.add_argument("--dense-arm", action="store_true",
                     help="--config fidasun: also time the dense fp16 plan of equal size now (time-limited process)")
     ap.add_argument("--prefill-tokens", type=int, default=8192,
@@ -784,10 +791,14 @@ def run_b200(args):
     elif c["kind"] == "hybrid":
         if cx.world != 1:
             raise SystemExit(f"--config {cfgname} is a single-GPU configuration")
-        from vllm_rs_b200 import _lib, bench_gibevik, bench_hybrid, bench_tasadra, bench_zalalix, bench_zufulix
+        from vllm_rs_b200 import (_lib, bench_gibevik, bench_hybrid, bench_sonalix, bench_tasadra, bench_zalalix,
+                                  bench_zufulix)
         launches0 = _lib.lib().b200_launch_count()
         with ClockSampler(cx.local) as clk:
-            if cfgname == "zufulix":
+            if cfgname == "sonalix":
+                sizes = [bench_sonalix.run(sz, layers=args.layers or 4, prefill=4096, batch=args.batch, ctx=2048,
+                                           reps=max(args.steps // 4, 3)) for sz in args.size.split(",")]
+            elif cfgname == "zufulix":
                 sizes = [bench_zufulix.run(sz, layers=args.layers or 4, prefill=4096, batch=args.batch, ctx=2048,
                                            reps=max(args.steps // 4, 3)) for sz in args.size.split(",")]
             elif cfgname == "tasadra":

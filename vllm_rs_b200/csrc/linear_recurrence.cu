@@ -476,17 +476,15 @@ decay_attn_kernel(float* __restrict__ out, const float* __restrict__ q, const fl
       cp_async_wait<0>();
     }
     __syncthreads();
-    // activation and scales of the pass, in place
-    if (act || q_scale != 1.f || k_scale != 1.f) {
+    // activation of the pass, in place
+    if (act) {
       for (int e = threadIdx.x; e < n * dim; e += kScanThreads) {
         const int r = e / dim, i = at(e - r * dim);
-        const float kv = ks[buf][r][i], qv = qs[buf][r][i];
-        ks[buf][r][i] = (act ? silu_exact(kv) : kv) * k_scale;
-        qs[buf][r][i] = (act ? silu_exact(qv) : qv) * q_scale;
+        ks[buf][r][i] = silu_exact(ks[buf][r][i]);
+        qs[buf][r][i] = silu_exact(qs[buf][r][i]);
       }
-      if (act)
-        for (int e = threadIdx.x; e < n * kScanCols; e += kScanThreads)
-          vs[buf][e / kScanCols][e % kScanCols] = silu_exact(vs[buf][e / kScanCols][e % kScanCols]);
+      for (int e = threadIdx.x; e < n * kScanCols; e += kScanThreads)
+        vs[buf][e / kScanCols][e % kScanCols] = silu_exact(vs[buf][e / kScanCols][e % kScanCols]);
       __syncthreads();
     }
     for (int r = 0; r < n; r += UN) {      // n is the same in every thread: the guards below do not diverge
@@ -499,7 +497,7 @@ decay_attn_kernel(float* __restrict__ out, const float* __restrict__ q, const fl
           load_seg(kr, &ks[buf][r + u][part * SEG]);
           load_seg(qr, &qs[buf][r + u][part * SEG]);
           if (CHAN) load_seg(ar, &as[buf][r + u][part * SEG]);
-          const float vv = vs[buf][r + u][threadIdx.x / RS];
+          const float vv = vs[buf][r + u][threadIdx.x / RS] * k_scale;      // (s k) v^T = k (s v)^T: one factor, not `dim`
           float y0 = 0.f, y1 = 0.f;
 #pragma unroll
           for (int j = 0; j < NR; j += 2) {
@@ -510,7 +508,7 @@ decay_attn_kernel(float* __restrict__ out, const float* __restrict__ q, const fl
               y1 += qr[j + 1] * s[j + 1];
             }
           }
-          y[u] = y0 + y1;
+          y[u] = (y0 + y1) * q_scale;
         }
       }
 #pragma unroll

@@ -329,6 +329,35 @@ def resid_rmsnorm(x, w, eps, w_offset=0.0, dtype=torch.bfloat16):
     return out
 
 
+def rmsnorm_rows(x, n, w, eps, w_offset=0.0, dtype=torch.bfloat16):
+    """RMS norm of the first n entries of every row of x fp32 [T, >= n]."""
+    _cuda(x, w)
+    out = torch.empty(x.shape[0], n, dtype=dtype, device=x.device)
+    _lib.lib().b200_rmsnorm_rows(_p(out), _p(x), x.shape[1], _p(w), x.shape[0], int(n), float(eps), float(w_offset),
+                                 _dt(dtype), _stream())
+    _lib.check()
+    return out
+
+
+def gate_rows(x, gate, dtype=torch.bfloat16):
+    """x fp32 [T, n] times the sigmoid of the first n entries of the rows of gate fp32 [T, >= n]."""
+    _cuda(x, gate)
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    _lib.lib().b200_gate_rows(_p(out), _p(x), _p(gate), gate.shape[1], x.shape[0], x.shape[1], _dt(dtype), _stream())
+    _lib.check()
+    return out
+
+
+def rotary_rows(x, rot_freq, positions, *, heads, dim, rot_half=True, rot_mag=1.0):
+    """The first 2 len(rot_freq) entries of the first `heads` heads (of `dim` entries) of every row of x fp32 [T, >= heads dim]
+    turn by position * rot_freq, in place."""
+    _cuda(x, rot_freq, positions)
+    _lib.lib().b200_rotary_rows(_p(x), x.shape[1], _p(rot_freq), float(rot_mag), int(bool(rot_half)), _p(positions),
+                                x.shape[0], int(heads), int(dim), 2 * rot_freq.numel(), _stream())
+    _lib.check()
+    return x
+
+
 def gated_group_norm(y, gate, w, group, eps, gate_first, dtype=torch.bfloat16, gate_act="silu"):
     """y, gate fp32 [T, C]; groups of `group` channels; w fp32 [C] or [group] (shared by the groups) or None;
     gate_act: "silu" or "sigmoid"."""
@@ -365,6 +394,22 @@ def latent_prep_queries(q, rot_freq, rot_mag, positions, *, heads, dim, rot_dim,
     q_full = torch.zeros(T, heads, kv_rank + rot_dim, dtype=torch.float32, device=q.device)
     _lib.lib().b200_latent_prep_queries(_p(q), q.shape[1], _p(q_plain), _p(q_full), _p(rot_freq), float(rot_mag),
                                         _p(positions), T, heads, dim, rot_dim, rot_dims, kv_rank, _dt(dtype), _stream())
+    _lib.check()
+    return q_plain, q_full
+
+
+def latent_prep_ex(q, low, cache, latent_norm_w, rot_freq, rot_mag, positions, slot_mapping, *, heads, dim, rot_dim,
+                   rot_dims, kv_rank, eps, rot_half=True):
+    """latent_prep with the queries fp32 [T, heads (dim + rot_dim)] and the raw latent rows fp32 [T, kv_rank + rot_dim + ..]
+    in different tensors, and a choice of rotary pairs."""
+    _cuda(q, low, cache, latent_norm_w, rot_freq, positions, slot_mapping)
+    T = q.shape[0]
+    q_plain = torch.empty(T, heads, dim, dtype=cache.dtype, device=q.device)
+    q_full = torch.zeros(T, heads, kv_rank + rot_dim, dtype=torch.float32, device=q.device)
+    _lib.lib().b200_latent_prep_ex(_p(q), q.shape[1], _p(low), low.shape[1], _p(q_plain), _p(q_full), _p(cache),
+                                   _p(latent_norm_w), _p(rot_freq), float(rot_mag), int(bool(rot_half)), _p(positions),
+                                   _p(slot_mapping), T, heads, dim, rot_dim, rot_dims, kv_rank, float(eps),
+                                   _dt(cache.dtype), _stream())
     _lib.check()
     return q_plain, q_full
 
@@ -468,52 +513,59 @@ def moe_route_ex(logits, bias, top, scale=1.0, groups=0, keep=0):
 
 
 def moe_route_full(logits, bias, top, scale=1.0, groups=0, keep=0, score="softmax", group_top=1, renorm=False):
-    """The router with every option: score "softmax" or "sigmoid", groups ranked by the sum of their `group_top` (1 or 2)
+    """The router with every option: score "softmax", "sigmoid" or "chosen" (logit + bias, softmax over the chosen), groups ranked by the sum of their `group_top` (1 or 2)
     best choice scores, chosen weights divided by their sum (renorm); see b200_moe_route_full."""
     _cuda(logits, bias)
     T, E = logits.shape
     idx = torch.empty(T, top, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, top, dtype=torch.float32, device=logits.device)
     _lib.lib().b200_moe_route_full(_p(logits), _p(bias), T, E, int(top), int(groups), int(keep),
-                                   {"softmax": 0, "sigmoid": 1}[score], int(group_top), int(bool(renorm)), float(scale),
+                                   {"softmax": 0, "sigmoid": 1, "chosen": 2}[score], int(group_top), int(bool(renorm)), float(scale),
                                    _p(idx), _p(w), _stream())
     _lib.check()
     return idx, w
 
 
-def moe_experts_rows(h, top_idx, w_up, w_down, *, act="silu_gate"):
+def _expert_act(act, limit, alpha, up_add):
+    return _lib.ExpertAct(kind={"silu_gate": 0, "relu2": 1, "clamped": 2}[act], limit=float(limit), alpha=float(alpha),
+                          up_add=float(up_add))
+
+
+def moe_experts_rows(h, top_idx, w_up, w_down, *, act="silu_gate", limit=0.0, alpha=1.0, up_add=0.0):
     """The chosen experts' output rows, unsummed: (rows fp32 [T * top, D] in bucket order, i32 [T * top]: the row of pair
-    token * top + choice)."""
+    token * top + choice).  act as in moe_experts_ex."""
     _cuda(h, top_idx, w_up, w_down)
     T, D = h.shape
     E, rows, _ = w_up.shape
-    F = rows // 2 if act == "silu_gate" else rows
+    F = rows if act == "relu2" else rows // 2
     top = top_idx.shape[1]
     nbytes = _lib.lib().b200_moe_workspace_bytes(T, E, top, D, F)
     ws = torch.empty(nbytes, dtype=torch.uint8, device=h.device)
     down, slot = C.c_void_p(), C.c_void_p()
-    _lib.lib().b200_moe_experts_rows(_p(h), _p(top_idx), _p(w_up), _p(w_down), T, E, top, D, F,
-                                     {"silu_gate": 0, "relu2": 1}[act], _dt(h.dtype), _p(ws), C.byref(down), C.byref(slot),
-                                     _stream())
+    _lib.lib().b200_moe_experts_rows_act(_p(h), _p(top_idx), _p(w_up), _p(w_down), T, E, top, D, F,
+                                         C.byref(_expert_act(act, limit, alpha, up_add)), _dt(h.dtype), _p(ws),
+                                         C.byref(down), C.byref(slot), _stream())
     _lib.check()
     at, base = lambda p, n, dt: ws[p.value - base:p.value - base + n * 4].view(dt), ws.data_ptr()
     return at(down, T * top * D, torch.float32).reshape(T * top, D), at(slot, T * top, torch.int32)
 
 
-def moe_experts_ex(out, h, top_idx, top_w, w_up, w_down, *, act="silu_gate", identity=0, accumulate=True, ident=None):
+def moe_experts_ex(out, h, top_idx, top_w, w_up, w_down, *, act="silu_gate", identity=0, accumulate=True, ident=None,
+                   limit=0.0, alpha=1.0, up_add=0.0):
     """out fp32 [T, D] (+)= the chosen experts of h [T, D]; act "silu_gate": w_up [E, 2 F, D]; "relu2": w_up [E, F, D];
+    "clamped": w_up [E, 2 F, D], the gated activation with the constants limit, alpha, up_add (b200_expert_act);
     indices >= E are identity experts and return the rows of `ident` (fp32 or h's dtype; default h)."""
     ident = h if ident is None else ident
     _cuda(out, h, top_idx, top_w, w_up, w_down, ident)
     T, D = out.shape
     E, rows, _ = w_up.shape
-    F = rows // 2 if act == "silu_gate" else rows
+    F = rows if act == "relu2" else rows // 2
     top = top_idx.shape[1]
     nbytes = _lib.lib().b200_moe_workspace_bytes(T, E + identity, top, D, F)
     ws = torch.empty(nbytes, dtype=torch.uint8, device=out.device)
-    _lib.lib().b200_moe_experts_ex(_p(out), _p(h), _p(top_idx), _p(top_w), _p(w_up), _p(w_down), T, E, int(identity), top,
-                                   D, F, {"silu_gate": 0, "relu2": 1}[act], int(bool(accumulate)), _p(ident),
-                                   int(ident.dtype == torch.float32), _dt(h.dtype), _p(ws), _stream())
+    _lib.lib().b200_moe_experts_act(_p(out), _p(h), _p(top_idx), _p(top_w), _p(w_up), _p(w_down), T, E, int(identity), top,
+                                    D, F, C.byref(_expert_act(act, limit, alpha, up_add)), int(bool(accumulate)), _p(ident),
+                                    int(ident.dtype == torch.float32), _dt(h.dtype), _p(ws), _stream())
     _lib.check()
     return out
 
