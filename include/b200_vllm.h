@@ -1039,7 +1039,8 @@ typedef struct b200_hybrid_layer {
   const void* dist_slopes;                  /* fp32 [heads] or NULL */
   int32_t shared_cache;                     /* latent attention: != 0: no latent projection of its own; kv_cache is
                                                another (earlier) layer's cache, which this layer only reads */
-  int32_t expert_act, shared_act;           /* expert_act: B200_EXPERT_*; shared_act 0: SiLU(gate) * up ([gate | up] rows); 1: relu(up)^2 (up rows only);
+  int32_t expert_act, shared_act;           /* expert_act: B200_EXPERT_*; shared_act 0: SiLU(gate) * up ([gate | up]
+                                               rows); 1: relu(up)^2 (up rows only);
                                                2 (shared_act): the exact GELU of up (up rows only) */
   int32_t identity_experts;                 /* router outputs experts .. experts + identity_experts - 1 return the input */
   int32_t route_groups, route_keep;         /* see b200_moe_route_ex (0: no groups) */

@@ -311,7 +311,10 @@ __global__ void hyper_step_kernel(const HyperArgs a) {
   float* u = sm + ((36 + S * S + 2 * S + 2 * a.top + 3) & ~3);
   const size_t t = a.rows ? a.rows[r] : r;
   const bool update = a.y != nullptr || a.down != nullptr;
-  for (int i = threadIdx.x; i < S * S; i += blockDim.x) mix[i] = update ? (a.mix ? a.mix[i] : (i % (S + 1) == 0 ? 1.f : 0.f)) : 0.f;
+  for (int i = threadIdx.x; i < S * S; i += blockDim.x) {
+    const float m = a.mix ? a.mix[i] : (i % (S + 1) == 0 ? 1.f : 0.f);
+    mix[i] = update ? m : 0.f;
+  }
   for (int i = threadIdx.x; i < S; i += blockDim.x) {
     ow[i] = update ? (a.out_w ? a.out_w[i] : 1.f) : 0.f;
     iw[i] = a.in_w ? a.in_w[i] : 1.f;
